@@ -46,6 +46,7 @@ ARCH_KEMIRAX = 100          # Info.version of the config.json-described families
 ARCH_DEGAVIK = 101
 ARCH_ZUFULIX = 102
 ARCH_PASOPEL = 103
+ARCH_PANUPEL = 104
 
 
 class B200Error(RuntimeError):

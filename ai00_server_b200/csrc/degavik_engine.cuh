@@ -117,10 +117,11 @@ void b200rwkv_engine::dg_load(const StFile& st, KxSizes& z) {
         const int H_ = c.heads, G_ = c.kv_heads, dk = c.dim, dv = c.vdim;
         REQUIRE(dv <= 1024, B200RWKV_ERR_UNSUPPORTED, "vdim must be <= 1024");
         if (c.mixer == KX_RETENTION || c.mixer == KX_DELTA) {
-            REQUIRE(std::max(retention_smem_bytes(dk, dv), delta_rule_smem_bytes(dk, dv)) <= 200 * 1024, B200RWKV_ERR_UNSUPPORTED,
-                    "head state too large for shared memory");
-            l.rec_state = (float*)dalloc((size_t)S * H_ * dk * dv * 4);
-            l.fixed.push_back({l.rec_state, (size_t)H_ * dk * dv});
+            REQUIRE(c.mixer == KX_DELTA || retention_smem_bytes(dk, dv) <= 200 * 1024, B200RWKV_ERR_UNSUPPORTED, "head state too large for shared memory");
+            REQUIRE(c.mixer != KX_DELTA || dk <= SCAN_MAX_DK, B200RWKV_ERR_UNSUPPORTED, "dim must be <= 1024");
+            const size_t per_head = c.mixer == KX_DELTA ? scan_state_floats(dk, dv) : (size_t)dk * dv;
+            l.rec_state = (float*)dalloc((size_t)S * H_ * per_head * 4);
+            l.fixed.push_back({l.rec_state, (size_t)H_ * per_head});
         }
         if (c.mixer == KX_RETENTION) {
             std::vector<float> d(H_);
@@ -164,7 +165,7 @@ void b200rwkv_engine::dg_load(const StFile& st, KxSizes& z) {
             while (l.wa_gt > 1 && window_attn_smem(qb, l.c.heads, l.c.dim, l.c.vdim, l.wa_gt) > 160 * 1024) l.wa_gt = (l.wa_gt + 1) / 2;
         }
     CK(cudaFuncSetAttribute(retention_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    CK(cudaFuncSetAttribute(delta_rule_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    CK(cudaFuncSetAttribute(delta_scan_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     CK(cudaFuncSetAttribute(window_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     // the largest cluster the attention launch may ask for: what the device can co-schedule at this layer's shared memory
     m.max_split = 8;
@@ -230,18 +231,14 @@ void b200rwkv_engine::dg_enqueue_layer(cudaStream_t s, KxLayer& l, int rows, int
     } else if (c.mixer == KX_DELTA) {
         const int C_ = l.conv_C;
         ShortConvParams cp{m.pr, PN, m.cv, C_, l.conv_w, l.conv_tail, C_, c.taps, mv};
-        launch_k(short_conv_kernel, dim3(rows, cdiv(C_, 256)), dim3(256), 0, cp, KC_OTHER, s, prof);
-        if (c.taps > 1) launch_k(conv_commit_kernel, dim3(nslot_grid, cdiv(C_, 256)), dim3(256), 0, cp, KC_OTHER, s, prof);
+        kx_short_conv(s, prof, cp, rows, nslot_grid, decode);
         kx_lin(s, prof, lin(m.pr + C_ + H_, PN, l.a2, m.z, H_ * dk, H_ * dk, l.a_rank, LE_STORE, l.a2_b), rows, 1);
         kx_lin(s, prof, lin(m.pr + C_ + H_ + l.a_rank, PN, l.g2, m.gl, H_ * dv, H_ * dv, l.g_rank), rows, 1);
-        DeltaRuleParams dp{m.cv, m.cv + G_ * dk, m.cv + 2 * G_ * dk, C_, m.z, H_ * dk, m.pr + C_, PN, m.gl, H_ * dv, l.a_log, l.norm_w, l.rec_state,
-                           m.vout, H_ * dv, H_, G_, dk, dv, 1.f / sqrtf((float)dk), 1e-6f, m.cfg.eps, mv};
-        if (dk <= DR_REG_MAX_DK && dv <= DR_REG_MAX_DV) {
-            auto kern = dk <= 32 ? delta_rule_reg_kernel<32> : (dk <= 64 ? delta_rule_reg_kernel<64> : delta_rule_reg_kernel<128>);
-            launch_k(kern, dim3(H_, nslot_grid), dim3(rup(dv, 32)), 0, dp, KC_WKV, s, prof);
-        } else {
-            launch_k(delta_rule_kernel, dim3(H_, nslot_grid), dim3(rup(dv, 32)), delta_rule_smem_bytes(dk, dv), dp, KC_WKV, s, prof);
-        }
+        const ScanShape sh = scan_shape(dk, dv, 3, decode);
+        DeltaScanParams dp{m.cv, m.cv + G_ * dk, m.cv + 2 * G_ * dk, C_, m.z, H_ * dk, m.pr + C_, PN, l.a_log, l.rec_state, H_, G_, dk, dv,
+                           1.f / sqrtf((float)dk), 1e-6f, sh, {m.vout, H_ * dv, nullptr, m.gl, H_ * dv, l.norm_w, 0, H_, dv, m.cfg.eps, 1.f, 0, mv}};
+        launch_k(delta_scan_kernel<true>, dim3(H_ * sh.ncta, nslot_grid), dim3(sh.threads), sh.smem_floats() * 4, dp, KC_WKV, s, prof);
+        if (sh.ncta > 1) launch_k(head_norm_kernel, dim3(rows, cdiv(H_, 4)), dim3(128), 0, dp.norm, KC_LN, s, prof);
     } else {
         AttnPrepParams ap{m.pr, m.pr + H_ * dk, m.pr + H_ * dk + G_ * dk, PN, m.q, H_ * dk, l.cache, m.d_table, m.npages, m.page, l.qn_w, l.kn_w,
                           l.temp, l.freq_d, H_, G_, dk, dv, c.rot.dims, c.scale, m.cfg.eps, mv, m.sm};

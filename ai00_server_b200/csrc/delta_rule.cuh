@@ -1,25 +1,24 @@
-// Gated delta rule with a per-key-channel decay, and the short causal convolutions in front of it.
+// Gated delta rule, and the short causal convolutions in front of it.
 //
-// Per value head, with the [dk, dv] f32 state S, unit-length key k and query q (q also times dk^-1/2), a decay vector g in
-// (0, 1)^dk acting on the rows of S, and a write strength beta in (0, 1):
-//     S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q          (the read-out sees this token's write)
-//     g = exp(-exp(A_h) * softplus(z)),  z = low-rank projection + bias,  beta = sigmoid(b)
-// The read-out is divided by its root mean square over dv, times a weight vector shared by the heads, times sigmoid of a
-// low-rank gate.  Several value heads may share one key / query head (value head h uses head h / (H / G)).
+// Per value head, with the [dk, dv] f32 state S, unit-length key k and query q (q also times dk^-1/2), a decay g in (0, 1) (one
+// number per head, or one per key channel acting on the rows of S) and a write strength beta in (0, 1):
+//     S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q                (the read-out sees this token's write)
+//     g = exp(-exp(A_h) * softplus(z)),  z = projection + bias,  beta = sigmoid(b)
+// The read-out is divided by its root mean square over dv, times a weight vector shared by the heads, times a gate (sigmoid or
+// silu of a projection).  Several value heads may share one key / query head (value head h uses head h / (H / G)).
 //
 //   short_conv_kernel     y[t, c] = silu(sum_j w[c, j] x[t - (taps - 1) + j, c]): per-channel causal convolution over time, the
 //                         last column is the current token's; inputs before the step come from the sequence's tail rows
 //                         (the last taps - 1 inputs, zeros at the start of a sequence)
 //   conv_commit_kernel    the step's last taps - 1 inputs become the sequence's new tail rows (own launch: every token of the
 //                         step has read the old tail by then)
-//   delta_rule_reg_kernel the state column of thread j in registers (dk <= 128, dv <= 256): the form that runs for usual head sizes
-//   delta_rule_kernel     one CTA per (value head, sequence of the step): the state sits in shared memory for the sequence's
-//                         tokens of this step, column j belongs to thread j (two passes over the column per token: decay +
-//                         S^T k, then update + read-out; no cross-thread traffic besides the unit norms and the output norm)
+//   short_conv_step_kernel   both at once for steps of one token per sequence
+//   delta_scan_kernel     the recurrence over the step's tokens of one sequence (state_scan.cuh)
 // Decays, logarithms, softplus, gates, unit norms, state and read-out are f32.
 #pragma once
 #include <cuda_runtime.h>
 #include "common.cuh"
+#include "state_scan.cuh"
 
 namespace b200 {
 
@@ -73,182 +72,143 @@ __global__ void __launch_bounds__(256) conv_commit_kernel(const ShortConvParams 
     }
 }
 
-struct DeltaRuleParams {
-    const float* q; const float* k; const float* v; int ld;      // conv outputs: q, k [T, G * dk], v [T, H * dv], row stride ld
-    const float* z; int ldz;                      // decay pre-activation [T, H * dk] (bias added)
-    const float* b; int ldb;                      // write-strength logits [T, H]
-    const float* gate; int ldgate;                // output-gate logits [T, H * dv]
-    const float* a_log;                           // [H]
-    const float* norm_w;                          // [dv]
-    float* state;                                 // [S][H][dk][dv] of this layer
-    float* out; int ldo;                          // [T, H * dv]
-    int H, G, dk, dv;
-    float q_scale, unit_eps, eps;
-    MetaView meta;
-};
-
-__host__ __device__ inline size_t delta_rule_smem_bytes(int dk, int dv) { return ((size_t)dk * dv + 3 * (size_t)dk + 64) * sizeof(float); }
-
-__global__ void delta_rule_kernel(const DeltaRuleParams p) {
-    const int h = blockIdx.x, si = blockIdx.y;
-    if (si >= p.meta.nslots()) return;
-    const int slot = p.meta.slot_id()[si], t0 = p.meta.slot_start()[si], nt = p.meta.slot_count()[si];
-    const int dk = p.dk, dv = p.dv, j = threadIdx.x, hk = h / (p.H / p.G);
-    const int nw = (blockDim.x + 31) >> 5;
-    extern __shared__ __align__(16) float dr_smem[];
-    float* S = dr_smem;                           // [dk][dv]
-    float* sq = S + (size_t)dk * dv;              // [dk]
-    float* sk = sq + dk;
-    float* sg = sk + dk;
-    float* red = sg + dk;                         // [2][32]
-    float* gS = p.state + ((size_t)slot * p.H + h) * dk * dv;
-    const int nst = dk * dv;
-    const bool vec = (nst % 4) == 0;
-    if (vec) {
-#pragma unroll 8
-        for (int e = j; e < nst / 4; e += blockDim.x) reinterpret_cast<float4*>(S)[e] = __ldg(reinterpret_cast<const float4*>(gS) + e);
-    } else {
-        for (int e = j; e < nst; e += blockDim.x) S[e] = gS[e];
-    }
-    const float rate = expf(p.a_log[h]);
-    for (int t = t0; t < t0 + nt; ++t) {
-        __syncthreads();
-        float qq = 0.f, kk = 0.f;
-        for (int i = j; i < dk; i += blockDim.x) {
-            const float qv = p.q[(size_t)t * p.ld + (size_t)hk * dk + i], kv = p.k[(size_t)t * p.ld + (size_t)hk * dk + i];
-            sq[i] = qv; sk[i] = kv;
-            qq = fmaf(qv, qv, qq); kk = fmaf(kv, kv, kk);
-            const float zz = p.z[(size_t)t * p.ldz + (size_t)h * dk + i];
-            const float sp = fmaxf(zz, 0.f) + log1pf(expf(-fabsf(zz)));      // softplus
-            sg[i] = expf(-rate * sp);
+// steps of one token per sequence: convolution and new tail in one pass (the thread that reads a channel's tail also moves it on)
+__global__ void __launch_bounds__(256) short_conv_step_kernel(const ShortConvParams p) {
+    const int t = blockIdx.x;
+    if (t >= p.meta.T()) return;
+    const int keep = p.taps - 1;
+    float* tl = p.tail + (size_t)p.meta.tok_slot()[t] * keep * p.C;
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < p.C; c += gridDim.y * blockDim.x) {
+        const float xv = p.x[(size_t)t * p.ldx + c];
+        float acc = 0.f;
+        for (int j = 0; j < keep; ++j) {
+            const float u = tl[(size_t)j * p.C + c];
+            acc = fmaf(p.w[(size_t)c * p.taps + j], u, acc);
+            if (j > 0) tl[(size_t)(j - 1) * p.C + c] = u;
         }
-#pragma unroll
-        for (int of = 16; of > 0; of >>= 1) { qq += __shfl_xor_sync(0xffffffffu, qq, of); kk += __shfl_xor_sync(0xffffffffu, kk, of); }
-        if ((j & 31) == 0) { red[j >> 5] = qq; red[32 + (j >> 5)] = kk; }
-        __syncthreads();
-        qq = 0.f; kk = 0.f;
-        for (int w = 0; w < nw; ++w) { qq += red[w]; kk += red[32 + w]; }
-        const float qn = p.q_scale / sqrtf(qq + p.unit_eps), kn = 1.f / sqrtf(kk + p.unit_eps);
-        const float bl = p.b[(size_t)t * p.ldb + h];
-        const float beta = 1.f / (1.f + expf(-bl));
-        float o = 0.f;
-        if (j < dv) {
-            const float vj = p.v[(size_t)t * p.ld + (size_t)h * dv + j];
-            float sk_dot = 0.f;
-            for (int i = 0; i < dk; ++i) {
-                const float s = sg[i] * S[(size_t)i * dv + j];
-                S[(size_t)i * dv + j] = s;
-                sk_dot = fmaf(s, sk[i] * kn, sk_dot);
-            }
-            const float u = beta * (vj - sk_dot);
-            for (int i = 0; i < dk; ++i) {
-                const float s = fmaf(sk[i] * kn, u, S[(size_t)i * dv + j]);
-                S[(size_t)i * dv + j] = s;
-                o = fmaf(s, sq[i] * qn, o);
-            }
-        }
-        float ss = j < dv ? o * o : 0.f;
-#pragma unroll
-        for (int of = 16; of > 0; of >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, of);
-        __syncthreads();                           // red has been read by every thread
-        if ((j & 31) == 0) red[j >> 5] = ss;
-        __syncthreads();
-        ss = 0.f;
-        for (int w = 0; w < nw; ++w) ss += red[w];
-        if (j < dv) {
-            const float gl = p.gate[(size_t)t * p.ldgate + (size_t)h * dv + j];
-            p.out[(size_t)t * p.ldo + (size_t)h * dv + j] = o / sqrtf(ss / (float)dv + p.eps) * p.norm_w[j] * (1.f / (1.f + expf(-gl)));
-        }
-    }
-    __syncthreads();
-    if (vec) {
-#pragma unroll 8
-        for (int e = j; e < nst / 4; e += blockDim.x) reinterpret_cast<float4*>(gS)[e] = reinterpret_cast<const float4*>(S)[e];
-    } else {
-        for (int e = j; e < nst; e += blockDim.x) gS[e] = S[e];
+        if (keep > 0) tl[(size_t)(keep - 1) * p.C + c] = xv;
+        acc = fmaf(p.w[(size_t)c * p.taps + keep], xv, acc);
+        p.y[(size_t)t * p.ldy + c] = p.silu ? acc / (1.f + expf(-acc)) : acc;
     }
 }
 
-// The same recurrence with the state column in REGISTERS (dk <= DKC <= 128, dv <= 256): thread j keeps S[0..dk)[j] for the whole
-// step, so the two passes over the column are straight-line FMAs on registers fed by broadcast reads of q, k and g from shared
-// memory (the shared-memory form above pays a load-after-store round trip per element).  Four partial sums shorten the
-// dependency chains of the two dot products.
-constexpr int DR_REG_MAX_DK = 128, DR_REG_MAX_DV = 256;
+struct DeltaScanParams {
+    const float* q; const float* k; const float* v; int ld;      // conv outputs: q, k [T, G * dk], v [T, H * dv], row stride ld
+    const float* z; int ldz;                      // decay pre-activation, bias added: [T, H * dk], or [T, H] with one decay per head
+    const float* b; int ldb;                      // write-strength logits [T, H]
+    const float* a_log;                           // [H]
+    float* state;                                 // [S][H] state records of this layer
+    int H, G, dk, dv;
+    float q_scale, unit_eps;
+    ScanShape s;                                  // rows = 3 (k, q, decays) with a decay per channel, else 2
+    HeadNormParams norm;                          // norm.x: raw read-outs, normed and gated in place
+};
 
-template <int DKC>
-__global__ void __launch_bounds__(DR_REG_MAX_DV) delta_rule_reg_kernel(const DeltaRuleParams p) {
-    const int h = blockIdx.x, si = blockIdx.y;
-    if (si >= p.meta.nslots()) return;
-    const int slot = p.meta.slot_id()[si], t0 = p.meta.slot_start()[si], nt = p.meta.slot_count()[si];
-    const int dk = p.dk, dv = p.dv, j = threadIdx.x, hk = h / (p.H / p.G);
-    const int nw = (blockDim.x + 31) >> 5;
-    __shared__ __align__(16) float sq[DKC], sk[DKC], sg[DKC];
-    __shared__ float red[64];
-    float* gS = p.state + ((size_t)slot * p.H + h) * dk * dv;
-    float s[DKC];
-#pragma unroll
-    for (int i = 0; i < DKC; ++i) s[i] = (i < dk && j < dv) ? gS[(size_t)i * dv + j] : 0.f;
-    const float rate = expf(p.a_log[h]);
-    for (int t = t0; t < t0 + nt; ++t) {
-        __syncthreads();
-        float qq = 0.f, kk = 0.f;
-        for (int i = j; i < DKC; i += blockDim.x) {
-            float qv = 0.f, kv = 0.f, gv = 1.f;
-            if (i < dk) {
-                qv = p.q[(size_t)t * p.ld + (size_t)hk * dk + i]; kv = p.k[(size_t)t * p.ld + (size_t)hk * dk + i];
-                const float zz = p.z[(size_t)t * p.ldz + (size_t)h * dk + i];
-                gv = expf(-rate * (fmaxf(zz, 0.f) + log1pf(expf(-fabsf(zz)))));
-            }
-            sq[i] = qv; sk[i] = kv; sg[i] = gv;
-            qq = fmaf(qv, qv, qq); kk = fmaf(kv, kv, kk);
+template <bool CHANNEL>
+__global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(const DeltaScanParams p) {
+    const ScanShape& sh = p.s;
+    const int h = blockIdx.x / sh.ncta, cb = blockIdx.x % sh.ncta, si = blockIdx.y;
+    const MetaView& meta = p.norm.meta;
+    if (si >= meta.nslots()) return;
+    const int slot = meta.slot_id()[si], t0 = meta.slot_start()[si], nt = meta.slot_count()[si];
+    const int dk = p.dk, dv = p.dv, hk = h / (p.H / p.G), ks = sh.ks;
+    const int x = threadIdx.x, warp = x >> 5, lane = x & 31, nw = blockDim.x >> 5;
+    const int part = x & (ks - 1), col = x >> sh.lks, j = cb * sh.cols + col, ncol = min(sh.cols, dv - cb * sh.cols);
+    extern __shared__ __align__(16) float scan_smem[];
+    const int krow = ks * SCAN_ROW, tokf = sh.tok_floats();
+    float* sbuf = scan_smem;                      // [nbuf][tc][k | q | (decays) | value entries]
+    float4* sscal = reinterpret_cast<float4*>(sbuf + (size_t)sh.nbuf * sh.tc * tokf);      // [tc] (decay, beta, 1 / |k|, q_scale / |q|)
+    float* sraw = reinterpret_cast<float*>(sscal + sh.tc);        // [nbuf][tc][2] decay and write-strength logits
+    float* rec = p.state + ((size_t)slot * p.H + h) * ((size_t)ks * sh.rt * dv);
+    float s[SCAN_R];
+    scan_load_state(sh, rec, dv, j, part, s);
+    for (int e = x; e < sh.nbuf * sh.tc * tokf; e += blockDim.x) sbuf[e] = 0.f;
+    __syncthreads();
+    auto stage = [&](int c) {
+        float* buf = sbuf + (size_t)(c % sh.nbuf) * sh.tc * tokf;
+        float* raw = sraw + (size_t)(c % sh.nbuf) * sh.tc * 2;
+        const int ta = t0 + c * sh.tc, n = min(sh.tc, nt - c * sh.tc);
+        scan_stage_keys(sh, buf, tokf, p.k + (size_t)ta * p.ld + (size_t)hk * dk, p.ld, n, dk);
+        scan_stage_keys(sh, buf + krow, tokf, p.q + (size_t)ta * p.ld + (size_t)hk * dk, p.ld, n, dk);
+        if (CHANNEL) scan_stage_keys(sh, buf + 2 * krow, tokf, p.z + (size_t)ta * p.ldz + (size_t)h * dk, p.ldz, n, dk);
+        scan_stage_cols(buf + sh.rows * krow, tokf, p.v + (size_t)ta * p.ld + (size_t)h * dv + cb * sh.cols, p.ld, n, ncol);
+        if (x < n) {
+            if (!CHANNEL) cp_async4(raw + 2 * x, p.z + (size_t)(ta + x) * p.ldz + h);
+            cp_async4(raw + 2 * x + 1, p.b + (size_t)(ta + x) * p.ldb + h);
         }
-#pragma unroll
-        for (int of = 16; of > 0; of >>= 1) { qq += __shfl_xor_sync(0xffffffffu, qq, of); kk += __shfl_xor_sync(0xffffffffu, kk, of); }
-        if ((j & 31) == 0) { red[j >> 5] = qq; red[32 + (j >> 5)] = kk; }
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+    };
+    const float rate = expf(p.a_log[h]);
+    const int nc = (nt + sh.tc - 1) / sh.tc;
+    stage(0);
+    for (int c = 0; c < nc; ++c) {
+        const int n = min(sh.tc, nt - c * sh.tc);
+        float* buf = sbuf + (size_t)(c % sh.nbuf) * sh.tc * tokf;
+        const float* raw = sraw + (size_t)(c % sh.nbuf) * sh.tc * 2;
+        if (sh.nbuf > 1 && c + 1 < nc) {
+            stage(c + 1);                          // into the buffer that group c - 1 used: everyone left it at the barrier below
+            asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        }
         __syncthreads();
-        qq = 0.f; kk = 0.f;
-        for (int w = 0; w < nw; ++w) { qq += red[w]; kk += red[32 + w]; }
-        const float qn = p.q_scale / sqrtf(qq + p.unit_eps), kn = 1.f / sqrtf(kk + p.unit_eps);
-        const float beta = 1.f / (1.f + expf(-p.b[(size_t)t * p.ldb + h]));
-        float o = 0.f;
-        if (j < dv) {
-            const float vj = p.v[(size_t)t * p.ld + (size_t)h * dv + j];
+        for (int t = warp; t < n; t += nw) {       // per token: lengths of k and q, decay, write strength
+            float* kr = buf + (size_t)t * tokf;
+            float kk = 0.f, qq = 0.f;
+            for (int i = lane; i < krow; i += 32) {
+                const float kv = kr[i], qv = kr[krow + i];
+                kk = fmaf(kv, kv, kk); qq = fmaf(qv, qv, qq);
+                if (CHANNEL) {
+                    const float z = kr[2 * krow + i];
+                    kr[2 * krow + i] = expf(-rate * (fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)))));
+                }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) { kk += __shfl_xor_sync(0xffffffffu, kk, o); qq += __shfl_xor_sync(0xffffffffu, qq, o); }
+            if (lane == 0) {
+                float g = 1.f;
+                if (!CHANNEL) {
+                    const float z = raw[2 * t];
+                    g = expf(-rate * (fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)))));
+                }
+                sscal[t] = make_float4(g, 1.f / (1.f + expf(-raw[2 * t + 1])), 1.f / sqrtf(kk + p.unit_eps), p.q_scale / sqrtf(qq + p.unit_eps));
+            }
+        }
+        __syncthreads();
+        float* orow = p.norm.x + (size_t)(t0 + c * sh.tc) * p.norm.ldx + (size_t)h * dv + j;
+        for (int t = 0; t < n; ++t) {
+            const float* kr = buf + (size_t)t * tokf + part * SCAN_ROW;
+            const float4 sc = sscal[t];
+            const float vj = buf[(size_t)t * tokf + sh.rows * krow + col];
             float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
 #pragma unroll
-            for (int i = 0; i < DKC; i += 4) {
-                s[i] *= sg[i]; s[i + 1] *= sg[i + 1]; s[i + 2] *= sg[i + 2]; s[i + 3] *= sg[i + 3];
-                d0 = fmaf(s[i], sk[i], d0); d1 = fmaf(s[i + 1], sk[i + 1], d1);
-                d2 = fmaf(s[i + 2], sk[i + 2], d2); d3 = fmaf(s[i + 3], sk[i + 3], d3);
+            for (int r = 0; r < SCAN_R; r += 4) {
+                const float4 k4 = *reinterpret_cast<const float4*>(kr + r);
+                if (CHANNEL) {
+                    const float4 g4 = *reinterpret_cast<const float4*>(kr + 2 * krow + r);
+                    s[r] *= g4.x; s[r + 1] *= g4.y; s[r + 2] *= g4.z; s[r + 3] *= g4.w;
+                } else {
+                    s[r] *= sc.x; s[r + 1] *= sc.x; s[r + 2] *= sc.x; s[r + 3] *= sc.x;
+                }
+                d0 = fmaf(s[r], k4.x, d0); d1 = fmaf(s[r + 1], k4.y, d1); d2 = fmaf(s[r + 2], k4.z, d2); d3 = fmaf(s[r + 3], k4.w, d3);
             }
-            const float u = beta * (vj - ((d0 + d1) + (d2 + d3)) * kn) * kn;       // u * kn: the write is k_unit u^T
+            const float d = scan_part_sum((d0 + d1) + (d2 + d3), ks);
+            const float u = sc.y * (vj - d * sc.z) * sc.z;         // u / |k|: the write is (k / |k|) u^T
             float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
 #pragma unroll
-            for (int i = 0; i < DKC; i += 4) {
-                s[i] = fmaf(sk[i], u, s[i]); s[i + 1] = fmaf(sk[i + 1], u, s[i + 1]);
-                s[i + 2] = fmaf(sk[i + 2], u, s[i + 2]); s[i + 3] = fmaf(sk[i + 3], u, s[i + 3]);
-                o0 = fmaf(s[i], sq[i], o0); o1 = fmaf(s[i + 1], sq[i + 1], o1);
-                o2 = fmaf(s[i + 2], sq[i + 2], o2); o3 = fmaf(s[i + 3], sq[i + 3], o3);
+            for (int r = 0; r < SCAN_R; r += 4) {
+                const float4 k4 = *reinterpret_cast<const float4*>(kr + r), q4 = *reinterpret_cast<const float4*>(kr + krow + r);
+                s[r] = fmaf(k4.x, u, s[r]); s[r + 1] = fmaf(k4.y, u, s[r + 1]); s[r + 2] = fmaf(k4.z, u, s[r + 2]); s[r + 3] = fmaf(k4.w, u, s[r + 3]);
+                o0 = fmaf(s[r], q4.x, o0); o1 = fmaf(s[r + 1], q4.y, o1); o2 = fmaf(s[r + 2], q4.z, o2); o3 = fmaf(s[r + 3], q4.w, o3);
             }
-            o = ((o0 + o1) + (o2 + o3)) * qn;
+            const float o = scan_part_sum((o0 + o1) + (o2 + o3), ks) * sc.w;
+            if (part == 0 && col < ncol) orow[(size_t)t * p.norm.ldx] = o;
         }
-        float ss = j < dv ? o * o : 0.f;
-#pragma unroll
-        for (int of = 16; of > 0; of >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, of);
-        __syncthreads();                           // red has been read by every thread
-        if ((j & 31) == 0) red[j >> 5] = ss;
         __syncthreads();
-        ss = 0.f;
-        for (int w = 0; w < nw; ++w) ss += red[w];
-        if (j < dv) {
-            const float gl = p.gate[(size_t)t * p.ldgate + (size_t)h * dv + j];
-            p.out[(size_t)t * p.ldo + (size_t)h * dv + j] = o / sqrtf(ss / (float)dv + p.eps) * p.norm_w[j] * (1.f / (1.f + expf(-gl)));
-        }
     }
-    if (j < dv) {
-#pragma unroll
-        for (int i = 0; i < DKC; ++i)
-            if (i < dk) gS[(size_t)i * dv + j] = s[i];
-    }
+    scan_store_state(sh, rec, dv, j, part, s);
+    if (sh.ncta == 1)
+        for (int t = warp; t < nt; t += nw) head_norm_row(p.norm, t0 + t, h, lane);
 }
 
 }  // namespace b200

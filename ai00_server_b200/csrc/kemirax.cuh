@@ -104,10 +104,14 @@ private:
 // ------------------------------------------------------------------------------------------------------------------
 // configuration
 // ------------------------------------------------------------------------------------------------------------------
-struct RotCfg { int dims = 0; double base = 10000.0; bool scaled = false; double factor = 1, original = 0, fast = 0, slow = 0; };
+struct RotCfg {
+    int dims = 0; double base = 10000.0;
+    bool scaled = false; double factor = 1, original = 0, fast = 0, slow = 0;          // ramp over the pairs (kx_rot_table)
+    bool banded = false; double low = 0, high = 0;                                     // bands of wavelengths (kx_rot_freqs), with factor and original
+};
 
-enum KxMixer { KX_LATENT = 0, KX_GLA = 1, KX_RETENTION = 2, KX_DELTA = 3, KX_WINDOW = 4, KX_BIASED = 5, KX_SINK = 6 };
-enum KxFamily { KX_FAMILY_KEMIRAX = 0, KX_FAMILY_DEGAVIK = 1, KX_FAMILY_ZUFULIX = 2, KX_FAMILY_PASOPEL = 3 };
+enum KxMixer { KX_LATENT = 0, KX_GLA = 1, KX_RETENTION = 2, KX_DELTA = 3, KX_WINDOW = 4, KX_BIASED = 5, KX_SINK = 6, KX_PARALLEL = 7 };
+enum KxFamily { KX_FAMILY_KEMIRAX = 0, KX_FAMILY_DEGAVIK = 1, KX_FAMILY_ZUFULIX = 2, KX_FAMILY_PASOPEL = 3, KX_FAMILY_PANUPEL = 4 };
 
 struct KxLayerCfg {
     int mixer = KX_LATENT;
@@ -129,6 +133,11 @@ struct KxLayerCfg {
     int pool = 0;                                                // tokens per block mean behind the window (0: none)
     int tensors_of = -1;                                         // index in the tensor names ("l<i>."); -1: the layer's own place
     int opens_pass = -1;                                         // >= 0: this run opens pass number `opens_pass` of the looped layers
+    // Panupel (panupel.cuh): attention (heads, kv_heads, dim, vdim, rot, scale above) beside a matrix memory; delta rule with one decay per head
+    bool head_decay = false;                                     // delta rule: one decay per head instead of one per key channel
+    int mm_heads = 0, mm_dim = 0, mm_vdim = 0;                   // matrix memory
+    float mm_cap = 0.f;                                          // its gates' pre-activations are squashed by cap * tanh(z / cap)
+    float attn_mul = 1.f, mm_mul = 1.f;                          // factors on the two sides' outputs
     int rot_dim = 0, kv_rank = 0, q_rank = 0, kv_from = -1;     // latent attention
     float scale = 1.f;
     RotCfg rot;
@@ -148,6 +157,7 @@ struct KxConfig {
     int streams = 0;                                             // copies of the residual (0: the plain residual)
     float embed_scale = 1.f;                                     // factor on the embedding row
     float logit_cap = 0.f;                                       // logits <- cap * tanh(logits / cap) (0: none)
+    float residual_mul = 1.f;                                    // factor on every sublayer's contribution to the residual
     bool has_loop = false;                                       // a run of layers is executed several times (`layers` lists every run)
     std::vector<KxLayerCfg> layers;
 };
@@ -155,6 +165,7 @@ struct KxConfig {
 static KxConfig dg_parse_config(const JVal& root);
 static KxConfig zf_parse_config(const JVal& root);
 static KxConfig ps_parse_config(const JVal& root);
+static KxConfig pn_parse_config(const JVal& root);
 
 // model registry of the families that come with a config.json: `architecture` names the design
 static KxConfig kx_parse_config(const char* json, size_t n) {
@@ -165,6 +176,7 @@ static KxConfig kx_parse_config(const char* json, size_t n) {
     if (arch == "Degavik") return dg_parse_config(root);
     if (arch == "Zufulix") return zf_parse_config(root);
     if (arch == "Pasopel") return ps_parse_config(root);
+    if (arch == "Panupel") return pn_parse_config(root);
     REQUIRE(arch == "Kemirax", B200RWKV_ERR_UNSUPPORTED, "config: unknown architecture '" + arch + "'");
     KxConfig c;
     c.vocab = root.integer("vocab");
@@ -236,6 +248,48 @@ static void kx_rot_table(const RotCfg& r, std::vector<float>& freq, float& mag) 
     }
 }
 
+// `loop` of a config: layers start .. stop - 1 are executed `times` times in a row.  The layer runs go to c.layers in execution
+// order; each names the layer of the file whose tensors it uses and, where it opens a pass, the number of that pass.
+static void kx_unroll_loop(const JVal& root, const std::vector<KxLayerCfg>& own, KxConfig& c) {
+    const int nl = (int)own.size();
+    int start = 0, stop = 0, times = 1;
+    if (root.has("loop")) {
+        const JVal& lp = root.at("loop");
+        start = lp.integer("start"); stop = lp.integer("stop"); times = lp.integer("times");
+        REQUIRE(start <= stop && stop <= nl && times >= 1, B200RWKV_ERR_INVALID, "config: loop must name layers start .. stop - 1 and times >= 1");
+        REQUIRE((long long)(stop - start) * times + nl <= 4096, B200RWKV_ERR_UNSUPPORTED, "config: too many layer runs");
+        c.has_loop = stop > start;
+    }
+    auto run = [&](int i, int opens) {
+        KxLayerCfg k = own[i];
+        k.tensors_of = i;
+        k.opens_pass = opens;
+        c.layers.push_back(k);
+    };
+    for (int i = 0; i < (c.has_loop ? start : nl); ++i) run(i, -1);
+    if (c.has_loop) {
+        for (int t = 0; t < times; ++t)
+            for (int i = start; i < stop; ++i) run(i, i == start ? t : -1);
+        for (int i = stop; i < nl; ++i) run(i, -1);
+    }
+}
+
+// rotary frequencies in double.  Banded: a pair whose wavelength is shorter than original / high keeps its frequency, one longer
+// than original / low turns `factor` times slower, and in between the two are blended linearly in original / wavelength
+static std::vector<double> kx_rot_freqs(const RotCfg& r) {
+    std::vector<double> f(std::max(r.dims / 2, 1), 0.0);
+    for (int i = 0; i < r.dims / 2; ++i) {
+        f[i] = std::pow(r.base, -2.0 * i / r.dims);
+        if (!r.banded) continue;
+        const double wave = 2.0 * M_PI / f[i];
+        if (wave < r.original / r.high) continue;
+        if (wave > r.original / r.low) { f[i] /= r.factor; continue; }
+        const double keep = (r.original / wave - r.low) / (r.high - r.low);
+        f[i] = (1.0 - keep) * f[i] / r.factor + keep * f[i];
+    }
+    return f;
+}
+
 // ------------------------------------------------------------------------------------------------------------------
 // device-side model
 // ------------------------------------------------------------------------------------------------------------------
@@ -283,6 +337,9 @@ struct KxLayer {
     int sa_qb = 1;                                               // tokens per chunk of the tile form in prompt steps
     int sa_hb_decode = 1;                                        // query heads per CTA in decode-shaped steps
     bool sa_reg = false;                                         // head sizes fit the register form of the attention kernel
+    // Panupel: norms on the sublayers' outputs, matrix memory
+    float *norm1b_w = nullptr, *norm2b_w = nullptr, *mm_norm_w = nullptr;
+    float *mm_state = nullptr, *mm_n = nullptr, *mm_m = nullptr;     // [S][H] x (state record of state_scan.cuh, dk floats, one float)
     // per-sequence memory of fixed size, in the order of the flat state record
     struct Block { float* base; size_t per_slot; };
     std::vector<Block> fixed;
@@ -304,6 +361,9 @@ struct SeqModel {
     float final_gain = 1.f;
     float* final_w = nullptr;                     // weight vector of the last norm (families that have one)
     float* final_b = nullptr;                     // its bias (layer-norm families)
+    __nv_bfloat16* pass_in = nullptr;             // [W][2 W] projection of (residual, embedding row) that opens a pass of a looped run of layers
+    cudaStream_t side_stream = nullptr;           // independent mixer halves run here beside the step's stream
+    cudaEvent_t side_fork = nullptr, side_join = nullptr;
     float* pass_vec = nullptr;                    // [passes][W] vector a looped run of layers adds when a pass begins
     int streams = 1;                              // copies of the residual a token row of x holds
     float* vfirst = nullptr;                      // [T, G * dv] values of the first blending attention layer, this step's tokens
@@ -328,6 +388,14 @@ struct SeqModel {
     int max_split = 16;
     int sa_ygroups = 1, sa_ygroups_decode = 1;    // head groups (grid rows) of the smallest windowed-attention launch of the model (prompt / decode shape)
     SeqMeta sm{nullptr, 0};
+    SeqModel() = default;
+    SeqModel(const SeqModel&) = delete;
+    SeqModel& operator=(const SeqModel&) = delete;
+    ~SeqModel() {
+        if (side_fork) cudaEventDestroy(side_fork);
+        if (side_join) cudaEventDestroy(side_join);
+        if (side_stream) cudaStreamDestroy(side_stream);
+    }
     size_t flat_floats(int ctx_rows) const;
     int max_D = 0;
 };

@@ -192,7 +192,8 @@ void b200rwkv_engine::kx_build(const StFile& st, const char* cfg_json, size_t cf
     m.W = m.cfg.width; m.V = m.cfg.vocab;
     const int W = m.W, nl = (int)m.cfg.layers.size();
     memset(&info, 0, sizeof(info));
-    info.version = m.cfg.family == KX_FAMILY_PASOPEL ? B200RWKV_ARCH_PASOPEL
+    info.version = m.cfg.family == KX_FAMILY_PANUPEL ? B200RWKV_ARCH_PANUPEL
+                   : m.cfg.family == KX_FAMILY_PASOPEL ? B200RWKV_ARCH_PASOPEL
                    : m.cfg.family == KX_FAMILY_ZUFULIX ? B200RWKV_ARCH_ZUFULIX
                    : (m.cfg.family == KX_FAMILY_DEGAVIK ? B200RWKV_ARCH_DEGAVIK : B200RWKV_ARCH_KEMIRAX); info.num_layer = nl; info.num_emb = W; info.num_vocab = m.V;
     L = nl; C = W; V = m.V; Vl = V; Cl = C; H = Hl = 0; N = 0; F = Fl = 0;
@@ -226,7 +227,8 @@ void b200rwkv_engine::kx_build(const StFile& st, const char* cfg_json, size_t cf
     for (int i = m.npages - 1; i >= 0; --i) m.free_pages.push_back(i);
 
     KxSizes z;
-    if (m.cfg.family == KX_FAMILY_PASOPEL) ps_load(st, z);
+    if (m.cfg.family == KX_FAMILY_PANUPEL) pn_load(st, z);
+    else if (m.cfg.family == KX_FAMILY_PASOPEL) ps_load(st, z);
     else if (m.cfg.family == KX_FAMILY_ZUFULIX) zf_load(st, z);
     else if (m.cfg.family == KX_FAMILY_DEGAVIK) dg_load(st, z);
     else kx_load(st, z);
@@ -305,6 +307,17 @@ void b200rwkv_engine::kx_lin(cudaStream_t s, Profiler* prof, LinParams p, int ro
     }
 }
 
+// the short convolutions of a layer: one launch in steps of one token per sequence, otherwise the convolution and then the new tails
+void b200rwkv_engine::kx_short_conv(cudaStream_t s, Profiler* prof, const ShortConvParams& cp, int rows, int nslot_grid, bool decode) {
+    const int cb = cdiv(cp.C, 256);
+    if (decode) {
+        launch_k(short_conv_step_kernel, dim3(rows, cb), dim3(256), 0, cp, KC_OTHER, s, prof);
+        return;
+    }
+    launch_k(short_conv_kernel, dim3(rows, cb), dim3(256), 0, cp, KC_OTHER, s, prof);
+    if (cp.taps > 1) launch_k(conv_commit_kernel, dim3(nslot_grid, cb), dim3(256), 0, cp, KC_OTHER, s, prof);
+}
+
 void b200rwkv_engine::kx_enqueue_step(cudaStream_t s, int rows, int rrows, bool decode, int nsplit, Profiler* prof) {
     launches_last_step = 0;
     SeqModel& m = *kx;
@@ -326,9 +339,11 @@ void b200rwkv_engine::kx_enqueue_step(cudaStream_t s, int rows, int rrows, bool 
         launch_k(embed_rows_kernel, dim3(rows), dim3(NORM_THREADS), 0, ep, KC_LN, s, prof);
     }
     const int nslot_grid = std::min(S, rows);
-    const bool own_stack = m.cfg.family == KX_FAMILY_ZUFULIX || m.cfg.family == KX_FAMILY_PASOPEL;    // these end with the last norm
+    // these end with the last norm
+    const bool own_stack = m.cfg.family == KX_FAMILY_ZUFULIX || m.cfg.family == KX_FAMILY_PASOPEL || m.cfg.family == KX_FAMILY_PANUPEL;
     if (m.cfg.family == KX_FAMILY_ZUFULIX) zf_enqueue_layers(s, rows, nslot_grid, decode, nsplit, prof);
     if (m.cfg.family == KX_FAMILY_PASOPEL) ps_enqueue_layers(s, rows, nslot_grid, decode, nsplit, prof);
+    if (m.cfg.family == KX_FAMILY_PANUPEL) pn_enqueue_layers(s, rows, nslot_grid, decode, nsplit, prof);
     for (size_t li = 0; li < m.layers.size() && !own_stack; ++li) {
         KxLayer& l = m.layers[li];
         const KxLayerCfg& c = l.c;
@@ -492,7 +507,7 @@ void b200rwkv_engine::kx_fill_step(int* hm, const std::vector<int>& slots, const
         int seen = 0;
         for (const KxLayer& l : m.layers) {
             if (l.c.mixer == KX_WINDOW) seen = std::max(seen, std::min(ctx_max, l.c.window + l.c.keep_first + QB));
-            if (l.c.mixer == KX_BIASED) seen = std::max(seen, ctx_max);
+            if (l.c.mixer == KX_BIASED || l.c.mixer == KX_PARALLEL) seen = std::max(seen, ctx_max);
             if (m.cfg.family == KX_FAMILY_PASOPEL)         // the window, and one row per block of older tokens
                 seen = std::max(seen, std::min(ctx_max, l.c.window + QB) + (l.c.pool > 0 ? ctx_max / l.c.pool : 0));
         }

@@ -77,28 +77,7 @@ static KxConfig ps_parse_config(const JVal& root) {
         }
         own.push_back(k);
     }
-    // the layer runs in execution order: layers before the loop, the looped layers once per pass, the rest
-    const int nl = (int)own.size();
-    int start = 0, stop = 0, times = 1;
-    if (root.has("loop")) {
-        const JVal& lp = root.at("loop");
-        start = lp.integer("start"); stop = lp.integer("stop"); times = lp.integer("times");
-        REQUIRE(start <= stop && stop <= nl && times >= 1, B200RWKV_ERR_INVALID, "config: loop must name layers start .. stop - 1 and times >= 1");
-        REQUIRE((long long)(stop - start) * times + nl <= 4096, B200RWKV_ERR_UNSUPPORTED, "config: too many layer runs");
-        c.has_loop = stop > start;
-    }
-    auto run = [&](int i, int opens) {
-        KxLayerCfg k = own[i];
-        k.tensors_of = i;
-        k.opens_pass = opens;
-        c.layers.push_back(k);
-    };
-    for (int i = 0; i < (c.has_loop ? start : nl); ++i) run(i, -1);
-    if (c.has_loop) {
-        for (int t = 0; t < times; ++t)
-            for (int i = start; i < stop; ++i) run(i, i == start ? t : -1);
-        for (int i = stop; i < nl; ++i) run(i, -1);
-    }
+    kx_unroll_loop(root, own, c);
     return c;
 }
 

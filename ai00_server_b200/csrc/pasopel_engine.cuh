@@ -5,70 +5,6 @@
 
 using namespace b200;
 
-typedef void (*SinkAttnKernel)(const SinkAttnParams);
-static inline SinkAttnKernel ps_attn_kernel(int rb) {
-    return rb >= 4 ? sink_attn_kernel<4> : (rb == 2 ? sink_attn_kernel<2> : sink_attn_kernel<1>);
-}
-
-// the attention launch sees every mixer as (H query heads, G key heads, key size, value size, value = leading part of the key?)
-struct PsAttnShape { int H, G, dk, dv; bool valias; };
-static inline PsAttnShape ps_attn_shape(const KxLayerCfg& c) {
-    if (c.mixer == KX_LATENT) return {c.heads, 1, c.kv_rank + c.rot_dim, c.kv_rank, true};        // absorbed form: one shared row
-    return {c.heads, c.kv_heads, c.dim, c.vdim, false};
-}
-
-// query heads per CTA: whole key heads, or a part of one key head's query heads; about `want`
-static inline int ps_heads_per_cta(int H, int G, int want) {
-    const int rep = H / G;
-    want = std::max(1, std::min(want, H));
-    if (G == 1) return want;
-    if (rep >= want) {
-        int d = want;
-        while (rep % d) --d;
-        return d;
-    }
-    return rep * (want / rep);
-}
-
-// the register form is built for key rows of one 512-byte piece per head.  (With three and five pieces, which the kernel's
-// template allows, a decode step of a 576-float latent row took 120 us where the tile form takes 84: every piece's loads wait
-// for the registers of the piece before it.)
-static inline SinkAttnKernel ps_attn_reg_kernel(int rb) {
-    return rb >= 4 ? sink_attn_reg_kernel<4, 1> : (rb == 2 ? sink_attn_reg_kernel<2, 1> : sink_attn_reg_kernel<1, 1>);
-}
-
-// how one attention launch of a layer runs: which kernel, its block size and shared memory, and the tile parameters
-struct PsAttnPlan { SinkAttnKernel kern; int threads; size_t smem; int gt, nbuf, qb, ks, hb; };
-
-static PsAttnPlan ps_attn_plan(const KxLayer& l, int qb_prompt, bool decode) {
-    const PsAttnShape a = ps_attn_shape(l.c);
-    const int rep = a.H / a.G, HB = decode ? l.sa_hb_decode : l.sa_hb;
-    const int nhc = std::min(rep, HB), ncv = HB / nhc;
-    PsAttnPlan p;
-    p.hb = HB;
-    if (l.sa_reg) {
-        const int qb = decode ? 1 : qb_prompt, rows = qb * nhc;              // rows of one key head in a full chunk
-        const int rb = rows >= 4 ? 4 : (rows >= 2 ? 2 : 1);
-        const int items = ncv * cdiv(rows, rb);
-        int ks = 1;                                // few items (decode): the 8 warps share each item's key tiles
-        while (ks < 8 && items * ks * 2 <= SAR_THREADS / 32) ks *= 2;
-        p.kern = ps_attn_reg_kernel(rb); p.threads = SAR_THREADS; p.smem = sink_attn_reg_smem(qb, HB, rep, a.dv, rb, ks);
-        p.gt = 1; p.nbuf = 1; p.qb = qb; p.ks = ks;
-        return p;
-    }
-    const int qb = decode ? 1 : l.sa_qb, rows = qb * nhc;
-    const int gt = decode ? l.sa_gt_decode : l.sa_gt, nbuf = decode ? l.sa_nbuf_decode : l.sa_nbuf;
-    // rows per warp: every key float a lane reads from the tile feeds one product per row, and the tile loop is bound by
-    // shared-memory reads, so as many rows as still leave 4 warps an item (8 in decode-shaped
-    int rb = SA_RB;
-    while (rb > 1 && std::min(gt, ncv) * cdiv(rows, rb) < (decode ? 8 : 4)) rb >>= 1;    // steps, whose CTAs have an SM to themselves)
-    p.kern = ps_attn_kernel(rb);
-    p.threads = std::min(gt, ncv) * cdiv(rows, rb) >= 16 ? SA_THREADS : 256;
-    p.smem = sink_attn_smem(qb, HB, a.dk, a.dv, gt, nbuf, a.valias);
-    p.gt = gt; p.nbuf = nbuf; p.qb = qb; p.ks = 1;
-    return p;
-}
-
 void b200rwkv_engine::ps_load(const StFile& st, KxSizes& z) {
     SeqModel& m = *kx;
     const int W = m.W, nr = (int)m.cfg.layers.size();
@@ -131,8 +67,7 @@ void b200rwkv_engine::ps_load(const StFile& st, KxSizes& z) {
                 l.ukT = kx_up16(t);
             }
             l.uv = kx_up16(kx_host_bf16(st, p + "mix.uv", (int64_t)H_ * dv, rk));
-            std::vector<double> fr(std::max(c.rot.dims / 2, 1), 0.0);
-            for (int f = 0; f < c.rot.dims / 2; ++f) fr[f] = std::pow(c.rot.base, -2.0 * f / c.rot.dims);
+            const std::vector<double> fr = kx_rot_freqs(c.rot);
             l.freq_d = (double*)dalloc(fr.size() * 8, false);
             CK(cudaMemcpy(l.freq_d, fr.data(), fr.size() * 8, cudaMemcpyHostToDevice));
         }
@@ -164,13 +99,12 @@ void b200rwkv_engine::ps_load(const StFile& st, KxSizes& z) {
     }
     // ---- the layer runs: the tensors of their layer, sequence memory of their own ----
     m.layers.resize(nr);
-    const int qb = 4;                              // tokens per chunk of a prompt step; a layer whose rows do not fit takes a part of a chunk per CTA
     for (int r = 0; r < nr; ++r) {
         KxLayer& l = m.layers[r];
         l = own[m.cfg.layers[r].tensors_of];
         l.c = m.cfg.layers[r];
         const KxLayerCfg& c = l.c;
-        const PsAttnShape a = ps_attn_shape(c);
+        const SaShape a = sa_shape(c);
         if (c.mixer == KX_SINK) {
             l.cache_D = a.G * (a.dk + a.dv);
             if (c.pool > 0) {
@@ -196,87 +130,8 @@ void b200rwkv_engine::ps_load(const StFile& st, KxSizes& z) {
                 if (c.has_shared) z.n_ys = std::max(z.n_ys, (size_t)c.sff);
             }
         }
-        // launch shape of the attention kernel: about 16 query heads per CTA, fewer (and then shorter chunks) where the rows of a
-        // chunk would not fit into shared memory beside one tile
-        // the register form takes key / value sizes that are multiples of four up to 128; longer rows (a latent) and odd sizes
-        // go through shared-memory tiles
-        l.sa_reg = a.dk % 4 == 0 && a.dv % 4 == 0 && l.cache_D % 4 == 0 && a.dk <= 128 && a.dv <= 128;
-        l.sa_hb = ps_heads_per_cta(a.H, a.G, 16);
-        l.sa_qb = qb;
-        // tile form: rows (tokens x heads) per CTA such that two CTAs fit an SM beside one tile each (one loads while the other
-        // multiplies); where that would leave fewer than four rows, one CTA per SM
-        const int hb0 = l.sa_hb;
-        for (size_t target : {(size_t)112 * 1024, (size_t)160 * 1024}) {
-            if (l.sa_reg) break;
-            l.sa_qb = qb; l.sa_hb = hb0;
-            while (sink_attn_smem(l.sa_qb, l.sa_hb, a.dk, a.dv, 1, 1, a.valias) > target) {
-                if (l.sa_qb > 1) l.sa_qb /= 2;
-                else if (l.sa_hb > 1 && ps_heads_per_cta(a.H, a.G, l.sa_hb / 2) < l.sa_hb) l.sa_hb = ps_heads_per_cta(a.H, a.G, l.sa_hb / 2);
-                else break;
-            }
-            if (sink_attn_smem(l.sa_qb, l.sa_hb, a.dk, a.dv, 1, 1, a.valias) <= target && l.sa_qb * l.sa_hb >= 4) break;
-        }
-        REQUIRE(l.sa_reg || sink_attn_smem(l.sa_qb, l.sa_hb, a.dk, a.dv, 1, 1, a.valias) <= 160 * 1024, B200RWKV_ERR_UNSUPPORTED,
-                "attention heads too large for shared memory");
     }
-    m.qb_prompt = qb;
-    m.sa_ygroups = m.sa_ygroups_decode = 1 << 30;
-    for (KxLayer& l : m.layers) {                  // as many key heads per tile load, and two tile buffers, where they fit
-        const PsAttnShape a = ps_attn_shape(l.c);
-        // decode-shaped steps have one row per head: the register form then takes one key head per CTA, so that a chunk's tiles
-        // are spread over more warps
-        l.sa_hb_decode = l.sa_reg ? ps_heads_per_cta(a.H, a.G, std::max(1, a.H / a.G)) : l.sa_hb;
-        m.sa_ygroups = std::min(m.sa_ygroups, cdiv(a.H, l.sa_hb));
-        m.sa_ygroups_decode = std::min(m.sa_ygroups_decode, cdiv(a.H, l.sa_hb_decode));
-        for (int dec = 0; dec < 2; ++dec) {
-            const int q = dec ? 1 : l.sa_qb;
-            const int hb = dec ? l.sa_hb_decode : l.sa_hb, ncv = std::max(1, hb / std::max(1, a.H / a.G));
-            int nbuf = 2, gt = ncv;
-            if (sink_attn_smem(q, hb, a.dk, a.dv, 1, 2, a.valias) > (size_t)(dec ? 200 : 112) * 1024) nbuf = 1;
-            while (gt > 1 && sink_attn_smem(q, hb, a.dk, a.dv, gt, nbuf, a.valias) > (dec ? 160 : 112) * 1024) gt = (gt + 1) / 2;
-            (dec ? l.sa_gt_decode : l.sa_gt) = gt;
-            (dec ? l.sa_nbuf_decode : l.sa_nbuf) = nbuf;
-        }
-    }
-    for (int rb = 1; rb <= SA_RB; rb *= 2) {
-        CK(cudaFuncSetAttribute(ps_attn_kernel(rb), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-        CK(cudaFuncSetAttribute(ps_attn_reg_kernel(rb), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    }
-    // the largest cluster the attention launch may ask for: what the device can co-schedule at this layer's shared memory
-    m.max_split = 8;
-    m.wa_ctas_prompt = m.wa_ctas_decode = 8;
-    for (const KxLayer& l : m.layers) {
-        const PsAttnPlan pp = ps_attn_plan(l, qb, false), pd = ps_attn_plan(l, qb, true);
-        REQUIRE(pp.smem <= 200 * 1024 && pd.smem <= 200 * 1024, B200RWKV_ERR_UNSUPPORTED, "attention heads too large for shared memory");
-        int cl = 8, cl_ok = 0;
-        for (; cl > 1; cl >>= 1) {
-            bool ok = true;
-            for (const PsAttnPlan* a : {&pp, &pd}) {
-                int lg = 0;
-                while ((1 << lg) < cl) ++lg;
-                cudaLaunchConfig_t cfg;
-                memset(&cfg, 0, sizeof(cfg));
-                cfg.gridDim = dim3(cl); cfg.blockDim = dim3(a->threads);
-                cfg.dynamicSmemBytes = a->smem;
-                cudaLaunchAttribute at;
-                at.id = cudaLaunchAttributeClusterDimension;
-                at.val.clusterDim.x = (unsigned)cl; at.val.clusterDim.y = 1; at.val.clusterDim.z = 1;
-                cfg.attrs = &at; cfg.numAttrs = 1;
-                int n = 0;
-                if (cudaOccupancyMaxActiveClusters(&n, a->kern, &cfg) != cudaSuccess || n <= 0) { ok = false; n = 0; }
-                cudaGetLastError();
-                int& cap = (a == &pd ? m.cl_cap_decode : m.cl_cap_prompt)[lg];      // clusters of this size the GPU holds at once
-                cap = std::min(cap, n);
-            }
-            if (ok && cl_ok == 0) cl_ok = cl;
-        }
-        m.max_split = std::min(m.max_split, std::max(cl_ok, 1));
-        int np = 1, nd = 1;
-        CK(cudaOccupancyMaxActiveBlocksPerMultiprocessor(&np, pp.kern, pp.threads, pp.smem));
-        CK(cudaOccupancyMaxActiveBlocksPerMultiprocessor(&nd, pd.kern, pd.threads, pd.smem));
-        m.wa_ctas_prompt = std::max(1, std::min(m.wa_ctas_prompt, np));
-        m.wa_ctas_decode = std::max(1, std::min(m.wa_ctas_decode, nd));
-    }
+    sa_plan_model(m);
     REQUIRE((size_t)W * 4 <= 200 * 1024, B200RWKV_ERR_UNSUPPORTED, "width too large for the norm kernel");
     CK(cudaFuncSetAttribute(pre_norm_kernel<NORM_THREADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     CK(cudaFuncSetAttribute(pre_norm_kernel<PRE_NORM_THREADS_FEW_ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
@@ -319,8 +174,8 @@ void b200rwkv_engine::ps_enqueue_layers(cudaStream_t s, int rows, int nslot_grid
         KxLayer& l = m.layers[li];
         const KxLayerCfg& c = l.c;
         const int H_ = c.heads, dv = c.vdim, PN = l.proj_n;
-        const PsAttnShape a = ps_attn_shape(c);
-        const PsAttnPlan plan = ps_attn_plan(l, m.qb_prompt, decode);
+        const SaShape a = sa_shape(c);
+        const SaPlan plan = sa_plan(l, m.qb_prompt, decode);
         boundary(nullptr, c.opens_pass > 0 ? m.embed : nullptr, c.opens_pass >= 0 ? m.pass_vec + (size_t)c.opens_pass * W : nullptr, l.norm1_w, m.h, 0,
                  nullptr);
         kx_lin(s, prof, lin(m.h, W, l.proj, m.pr, PN, PN, W, LE_STORE, l.proj_b), rows, 1);
@@ -329,14 +184,13 @@ void b200rwkv_engine::ps_enqueue_layers(cudaStream_t s, int rows, int nslot_grid
         sp.cache = l.cache; sp.table = m.d_table; sp.stride = m.npages; sp.page = m.page; sp.D = l.cache_D;
         sp.sink = l.sink; sp.H = a.H; sp.G = a.G; sp.dk = a.dk; sp.dv = a.dv; sp.HB = plan.hb; sp.win = c.window;
         sp.qb = plan.qb; sp.gt = plan.gt; sp.cl = nsplit; sp.nbuf = plan.nbuf; sp.valias = a.valias ? 1 : 0; sp.ks = plan.ks;
-        sp.nsub = decode ? 1 : m.qb_prompt / plan.qb;
+        sp.out_mul = 1.f; sp.nsub = decode ? 1 : m.qb_prompt / plan.qb;
         sp.meta = mv; sp.sm = m.sm;
         const dim3 attn_grid(chunks_grid * sp.nsub * nsplit, cdiv(a.H, plan.hb));
         if (c.mixer == KX_SINK) {
             const int G_ = c.kv_heads, dk = c.dim, C_ = l.conv_C;
             ShortConvParams cp{m.pr, PN, m.cv, C_, l.conv_w, l.conv_tail, C_, c.taps, mv, 0};
-            launch_k(short_conv_kernel, dim3(rows, cdiv(C_, 256)), dim3(256), 0, cp, KC_OTHER, s, prof);
-            if (c.taps > 1) launch_k(conv_commit_kernel, dim3(nslot_grid, cdiv(C_, 256)), dim3(256), 0, cp, KC_OTHER, s, prof);
+            kx_short_conv(s, prof, cp, rows, nslot_grid, decode);
             // unit-RMS queries (times the score scale) to the step buffer, unit-RMS keys and the keys as they are (the values) to the cache
             BiasAttnPrepParams ap{m.cv, m.cv + H_ * dk, m.cv + H_ * dk, C_, m.q, H_ * dk, l.cache, m.d_table, m.npages, m.page,
                                   m.vfirst, 0, BA_V_PLAIN, 0.f, H_, G_, dk, dv, c.scale, m.cfg.eps, mv, m.sm};

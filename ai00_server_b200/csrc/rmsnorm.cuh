@@ -9,7 +9,8 @@
 //   norm_add_kernel        x += y / rms(y) * w: the norm sits on a sublayer's output (optionally combining routed expert rows first)
 //   pre_norm_kernel        the boundary in front of a pre-norm sublayer in one pass: the routed experts that just finished are
 //                          combined into the residual, a looped run of layers that begins adds the embedding row and its pass
-//                          vector, and the normed row (or, at the end of the stack, the compact rows that want logits) is written
+//                          vector, and the normed row (or, at the end of the stack, the compact rows that want logits) is written;
+//                          where sublayers also have a norm on their output, that norm and the residual sum come first
 #pragma once
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -200,8 +201,10 @@ __global__ void __launch_bounds__(NORM_THREADS) norm_add_kernel(const NormAddPar
 
 // The boundary in front of a pre-norm sublayer.  In this order, each part optional:
 //   x[t] += sum_k wgt[t, k] rows[row_of[t, k]] + shared[t]     the routed feed-forward that just finished (its combine step)
+//   x[t] += post_mul * y[t] / rms(y[t]) * post_w               the sublayer that just finished, with a norm on its output
 //   snap[t] = x[t]                                             the residual as the finished layer leaves it (bring-up aid)
 //   x[t] += table[token[t]] + vec                              a pass of a looped run of layers begins
+//   cat[t] = [x[t]; table[token[t]]]                           a pass begins with a projection of both (then table adds nothing to x)
 //   h[t] = x[t] / rms(x[t]) * weight                           the sublayer's input; `weight` holds the whole factor (a model
 //                                                              that stores offsets from one uploads 1 + w)
 // With `compact` only the rows that want logits are normed and land in h[row]; `hidden` gets a copy of every residual row.
@@ -221,6 +224,10 @@ struct PreNormParams {
     float* hidden;            // [T, W] (nullptr: none)
     int W;
     MetaView meta;
+    const float* y = nullptr;         // [T, W] finished sublayer's output (nullptr: none)
+    const float* post_w = nullptr;    // [W]
+    float post_mul = 1.f;
+    float* cat = nullptr;             // [T, 2 W] (nullptr: none)
 };
 
 constexpr int PRE_NORM_THREADS_FEW_ROWS = 1024;    // block size for steps of few tokens (decode): a thread then owns one or two columns
@@ -240,10 +247,21 @@ __global__ void __launch_bounds__(THREADS) pre_norm_kernel(const PreNormParams p
             if (k < p.top) { rw[k] = p.row_of[(size_t)t * p.top + k]; wg[k] = p.wgt[(size_t)t * p.top + k]; }
     }
     const __nv_bfloat16* er = p.table ? p.table + (size_t)p.meta.tok()[t] * W : nullptr;
-    const bool writes = p.rows || er || p.vec;
-    float ss = 0.f;
+    const bool writes = p.rows || p.y || (er && !p.cat) || p.vec;
+    float ss = 0.f, post_r = 0.f;
+    if (p.y) {
+        for (int c = threadIdx.x; c < W; c += blockDim.x) {        // a thread meets the same columns again below
+            const float v = p.y[(size_t)t * W + c];
+            pre_norm_row[c] = v;
+            ss = fmaf(v, v, ss);
+        }
+        ss = rms_block_sum(ss, red);
+        post_r = p.post_mul / sqrtf(ss / (float)W + p.eps);
+        ss = 0.f;
+    }
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
         float v = xr[c];
+        if (p.y) v += pre_norm_row[c] * post_r * p.post_w[c];
         if (p.rows) {
             float f = 0.f;
 #pragma unroll
@@ -253,7 +271,12 @@ __global__ void __launch_bounds__(THREADS) pre_norm_kernel(const PreNormParams p
             v += f;
         }
         if (p.snap) p.snap[(size_t)t * W + c] = v;
-        if (er) v += __bfloat162float(er[c]);
+        if (p.cat) {
+            p.cat[(size_t)t * 2 * W + c] = v;
+            p.cat[(size_t)t * 2 * W + W + c] = er ? __bfloat162float(er[c]) : 0.f;
+        } else if (er) {
+            v += __bfloat162float(er[c]);
+        }
         if (p.vec) v += p.vec[c];
         if (writes) xr[c] = v;
         if (p.hidden) p.hidden[(size_t)t * W + c] = v;

@@ -1,6 +1,6 @@
 // Softmax attention over a paged cache with a sliding window, a learned "sink" term per head in the softmax denominator, and
 // (optionally) block means of the keys / values that have left the window.  No positions enter the scores here: a layer that
-// rotates its queries and keys does so before it calls this.
+// rotates its queries and keys does so before it calls this (rot_prep_kernel).
 //
 // H query heads, G key / value heads (query head h reads head h / (H / G)).  A cache row of D floats holds, for every key /
 // value head c, a key of dk floats at `koff + c dk` and a value of dv floats at `voff + c dv` (the two may be the same floats:
@@ -9,10 +9,12 @@
 //     blocks   b with  (b + 1) pool <= i - win + 1      (pool > 0): the mean of the cache rows b pool .. b pool + pool - 1,
 //              kept in a second pool of rows with the same layout (pool_write_kernel) so that a block costs one row to read
 //     s_h(i, u) = (q_h(i) . k(u)) * scale           over the visible tokens and blocks u together
-//     o_h(i) = sum_u exp(s_h(i, u)) v(u) / (exp(sink_h) + sum_u exp(s_h(i, u)))        * sigmoid(gate_h(i))  (gate optional)
+//     o_h(i) = sum_u exp(s_h(i, u)) v(u) / (exp(sink_h) + sum_u exp(s_h(i, u)))        * sigmoid(gate_h(i)) * out_mul
+// The gate is optional: one number per output entry, or one per head.
 //
 //   pool_write_kernel     every token of the step that closes a block writes the block's mean row (sums in position order, f32)
 //   pool_rebuild_kernel   the same for all closed blocks of one sequence (after a state import)
+//   rot_prep_kernel       queries and keys of a layer that norms the whole projection and rotates half against half
 //   sink_attn_kernel      a cluster of 1..8 CTAs per (chunk of consecutive tokens of one sequence, group of HB query heads);
 //                         the visible block rows and then the window's token rows form 32-key tiles that are dealt out among
 //                         the cluster's CTAs; every CTA walks its tiles once with a running maximum / sum per (token, head) row
@@ -28,6 +30,7 @@
 #include "common.cuh"
 #include "latent_attn.cuh"
 #include "linear.cuh"
+#include "rmsnorm.cuh"
 
 namespace b200 {
 
@@ -72,6 +75,60 @@ __global__ void __launch_bounds__(128) pool_rebuild_kernel(const PoolWriteParams
     if ((int)blockIdx.x < p.nblocks) sa_pool_block(p, p.table + (size_t)p.slot * p.stride, blockIdx.x);
 }
 
+// Queries and keys of an attention layer that norms each projection as a whole and rotates half against half: per token
+//     q <- rot(q / rms(q over all heads) * w_q) -> step buffer,   k <- rot(k / rms(k over all heads) * w_k) and v -> the cache row
+// where entry i of a head turns with entry i + dims / 2 (i < dims / 2) by position * freq[i] and entries from dims on stay.  One CTA
+// per token; the angles are formed and reduced in double, once per token.  Dynamic shared memory: dims floats.
+struct RotPrepParams {
+    const float* q; const float* k; const float* v; int ld;      // projection rows: q [H dk], k [G dk], v [G dv]
+    float* qo; int ldq;                            // [T, H dk]
+    float* cache;                                  // [pages][page][G dk + G dv]
+    const int* table; int stride, page;
+    const float* wq; const float* wk;              // [H dk], [G dk]
+    const double* freq;                            // [dims / 2]
+    int H, G, dk, dv, dims;
+    float eps;
+    MetaView meta; SeqMeta sm;
+};
+
+constexpr int ROT_PREP_THREADS = 256;
+
+__global__ void __launch_bounds__(ROT_PREP_THREADS) rot_prep_kernel(const RotPrepParams p) {
+    __shared__ float red[32];
+    extern __shared__ __align__(16) float rot_cs[];              // [dims / 2] cosines, [dims / 2] sines
+    const int t = blockIdx.x;
+    if (t >= p.meta.T()) return;
+    const int slot = p.meta.tok_slot()[t], ipos = p.sm.tok_pos()[t], half = p.dims >> 1;
+    float* row = p.cache + sa_token_row(p.table + (size_t)slot * p.stride, p.page, ipos) * (size_t)(p.G * (p.dk + p.dv));
+    for (int i = threadIdx.x; i < half; i += blockDim.x) rot_cos_sin(ipos, p.freq[i], rot_cs[i], rot_cs[half + i]);
+    const float* qs = p.q + (size_t)t * p.ld;
+    const float* ks = p.k + (size_t)t * p.ld;
+    const float* vs = p.v + (size_t)t * p.ld;
+    const int nq = p.H * p.dk, nk = p.G * p.dk;
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x; i < nq; i += blockDim.x) sq = fmaf(qs[i], qs[i], sq);
+    for (int i = threadIdx.x; i < nk; i += blockDim.x) sk = fmaf(ks[i], ks[i], sk);
+    sq = rms_block_sum(sq, red);
+    sk = rms_block_sum(sk, red);                   // its barriers also publish the angles
+    const float rq = 1.f / sqrtf(sq / (float)nq + p.eps), rk = 1.f / sqrtf(sk / (float)nk + p.eps);
+    for (int e = threadIdx.x; e < nq + nk; e += blockDim.x) {
+        const bool isq = e < nq;
+        const int o = isq ? e : e - nq, i = o % p.dk;
+        const float* src = isq ? qs : ks;
+        const float* w = isq ? p.wq : p.wk;
+        const float r = isq ? rq : rk;
+        float val = src[o] * r * w[o];
+        if (i < p.dims) {
+            const int f = i < half ? i : i - half, o2 = i < half ? o + half : o - half;
+            const float other = src[o2] * r * w[o2];
+            val = i < half ? val * rot_cs[f] - other * rot_cs[half + f] : val * rot_cs[f] + other * rot_cs[half + f];
+        }
+        if (isq) p.qo[(size_t)t * p.ldq + o] = val;
+        else row[o] = val;
+    }
+    for (int i = threadIdx.x; i < p.G * p.dv; i += blockDim.x) row[nk + i] = vs[i];
+}
+
 struct SinkAttnParams {
     const float* q; int ldq;                       // query of (t, h): q + t ldq + h dk
     const float* cache; const float* pcache;       // token rows; block-mean rows (nullptr / pool = 0: none)
@@ -79,6 +136,8 @@ struct SinkAttnParams {
     int D, koff, voff;
     float* out; int ldo;                           // [T, H dv]
     const float* gate; int ldg;                    // out *= sigmoid(gate[t ldg + h dv + d])   (nullptr: no gate)
+    int gate_heads;                                // the gate has one number per head: gate[t ldg + h]
+    float out_mul;                                 // factor on the output
     const float* sink;                             // [H] (nullptr: no sink term)
     float scale;
     int H, G, dk, dv, HB;                          // HB query heads per CTA: a multiple of H / G, or a divisor of it
@@ -347,8 +406,8 @@ __global__ void __launch_bounds__(SA_THREADS) sink_attn_kernel(const SinkAttnPar
             }
         }
         float o = num / den;
-        if (p.gate) o *= lin_sigmoid(p.gate[(size_t)t * p.ldg + (size_t)h * dv + d]);
-        p.out[(size_t)t * p.ldo + (size_t)h * dv + d] = o;
+        if (p.gate) o *= lin_sigmoid(p.gate[(size_t)t * p.ldg + (p.gate_heads ? (size_t)h : (size_t)h * dv + d)]);
+        p.out[(size_t)t * p.ldo + (size_t)h * dv + d] = o * p.out_mul;
     }
     cluster.sync();                                // nobody leaves while its shared memory is still being read
 }
@@ -604,8 +663,8 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
                 den = fmaf(lr[rk], f, den);
             }
         float o = num / den;
-        if (p.gate) o *= lin_sigmoid(p.gate[(size_t)t * p.ldg + (size_t)h * dv + d]);
-        p.out[(size_t)t * p.ldo + (size_t)h * dv + d] = o;
+        if (p.gate) o *= lin_sigmoid(p.gate[(size_t)t * p.ldg + (p.gate_heads ? (size_t)h : (size_t)h * dv + d)]);
+        p.out[(size_t)t * p.ldo + (size_t)h * dv + d] = o * p.out_mul;
     }
     cluster.sync();                                // nobody leaves while its shared memory is still being read
 }

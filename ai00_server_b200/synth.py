@@ -664,3 +664,93 @@ def make_pasopel(layers: list, width: int = 64, vocab: int = 96, eps: float = 1e
     bits = {k: to_bf16_bits(np.asarray(v, np.float32).reshape(np.shape(v))) for k, v in t.items()}
     rounded = {k: (b.astype(np.uint32) << 16).view(np.float32).reshape(np.shape(t[k])).astype(np.float64) for k, b in bits.items()}
     return json.dumps(cfg).encode(), pack_st_bf16(t), rounded
+
+
+# ----------------------------------------------------------------------------------------------------------------------
+# Panupel family (config.json + bf16 safetensors): random weights for tests and bench.py
+# ----------------------------------------------------------------------------------------------------------------------
+def panupel_layer(kind: str, *, heads=4, kv_heads=None, dim=16, vdim=None, conv=3, rot_dims=None, base=10000.0, scaling=None, scale=None,
+                  mm_heads=2, mm_dim=12, mm_vdim=None, gate_cap=15.0, left_scale=1.1, right_scale=0.8, ff=48) -> dict:
+    """One entry of config['layers'].  kind: 'parallel' | 'delta'; ff None: no feed-forward; scaling: (factor, low, high, original) or None."""
+    vdim = int(vdim or dim)
+    if kind == "parallel":
+        rot = {"base": float(base), "dims": int(dim if rot_dims is None else rot_dims)}
+        if scaling:
+            rot["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+        mixer = {"left": {"heads": heads, "kv_heads": int(kv_heads or heads), "dim": dim, "vdim": vdim, "rot": rot,
+                          "scale": float(scale if scale is not None else dim ** -0.5)},
+                 "right": {"heads": mm_heads, "dim": mm_dim, "vdim": int(mm_vdim or mm_dim), "gate_cap": float(gate_cap)},
+                 "left_scale": float(left_scale), "right_scale": float(right_scale)}
+    elif kind == "delta":
+        mixer = {"heads": heads, "kv_heads": int(kv_heads or heads), "dim": dim, "vdim": vdim, "conv": int(conv)}
+    else:
+        raise ValueError(kind)
+    return {"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": int(ff)} if ff else None}
+
+
+def make_panupel(layers: list, width: int = 64, vocab: int = 96, eps: float = 1e-5, seed: int = 0, loop: tuple | None = (0, 1, 2),
+                 residual_mult: float = 0.6, arrays: bool = True):
+    """(config.json bytes, safetensors image, dict of float64 arrays holding the bf16-rounded values, or None when `arrays` is
+    off) for a random model of the family.  loop: (start, stop, times) or None."""
+    rng = np.random.default_rng(seed)
+    W = width
+    t = {}
+
+    def mat(n, k, g=1.0):
+        return (rng.standard_normal((n, k)) * (g / np.sqrt(k))).astype(np.float32)
+
+    def norm(name, n=W):
+        t[name] = rng.uniform(0.5, 1.5, n).astype(np.float32)
+
+    t["embed"] = rng.standard_normal((vocab, W)).astype(np.float32)
+    if loop is not None:
+        t["loop.in"] = mat(W, 2 * W)
+    for i, l in enumerate(layers):
+        p, m = "l%d." % i, l["mixer"]
+        norm(p + "norm1")
+        norm(p + "norm1b")
+        if l["type"] == "delta":
+            H, G, dk, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            for n, rows in (("q", G * dk), ("k", G * dk), ("v", H * dv)):
+                t[p + "mix." + n] = mat(rows, W, 2.0)
+                t[p + "mix." + n + ".conv"] = (rng.standard_normal((rows, m["conv"])) * 0.6).astype(np.float32)
+            t[p + "mix.b"] = mat(H, W, 2.0)
+            t[p + "mix.a"] = mat(H, W, 2.0)
+            t[p + "mix.A_log"] = rng.uniform(-4.0, 0.0, H).astype(np.float32)
+            t[p + "mix.dt_bias"] = rng.uniform(-4.0, 1.0, H).astype(np.float32)
+            t[p + "mix.norm"] = rng.uniform(0.5, 1.5, dv).astype(np.float32)
+            t[p + "mix.g"] = mat(H * dv, W, 2.0)
+            t[p + "mix.o"] = mat(W, H * dv)
+        else:
+            a, b = m["left"], m["right"]
+            H, G, dk, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            q = p + "mix.left."
+            t[q + "q"], t[q + "k"], t[q + "v"] = mat(H * dk, W), mat(G * dk, W), mat(G * dv, W)
+            norm(q + "q.norm", H * dk)
+            norm(q + "k.norm", G * dk)
+            t[q + "sink"] = rng.standard_normal(H).astype(np.float32)
+            t[q + "g"] = mat(H, W, 2.0)
+            t[q + "o"] = mat(W, H * dv)
+            H, dk, dv = b["heads"], b["dim"], b["vdim"]
+            q = p + "mix.right."
+            t[q + "q"], t[q + "k"], t[q + "v"], t[q + "g"] = mat(H * dk, W, 1.5), mat(H * dk, W, 1.5), mat(H * dv, W), mat(H * dv, W, 2.0)
+            norm(q + "norm", H * dv)
+            t[q + "i"], t[q + "f"] = mat(H, W, 2.0), mat(H, W, 2.0)
+            t[q + "i.b"] = rng.uniform(-3.0, 1.0, H).astype(np.float32)
+            t[q + "f.b"] = rng.uniform(0.0, 6.0, H).astype(np.float32)
+            t[q + "o"] = mat(W, H * dv)
+        f = l.get("mlp")
+        if f:
+            norm(p + "norm2")
+            norm(p + "norm2b")
+            t[p + "mlp.gate"], t[p + "mlp.up"], t[p + "mlp.down"] = mat(f["ff"], W, 2.0), mat(f["ff"], W, 2.0), mat(W, f["ff"])
+    norm("final.norm")
+    t["head"] = mat(vocab, W)
+    cfg = {"architecture": "Panupel", "layers": layers, "norm": {"eps": eps}, "residual_mult": float(residual_mult), "vocab": vocab, "width": W}
+    if loop is not None:
+        cfg["loop"] = {"start": int(loop[0]), "stop": int(loop[1]), "times": int(loop[2])}
+    if not arrays:
+        return json.dumps(cfg).encode(), pack_st_bf16(t), None
+    bits = {k: to_bf16_bits(np.asarray(v, np.float32).reshape(np.shape(v))) for k, v in t.items()}
+    rounded = {k: (b.astype(np.uint32) << 16).view(np.float32).reshape(np.shape(t[k])).astype(np.float64) for k, b in bits.items()}
+    return json.dumps(cfg).encode(), pack_st_bf16(t), rounded
