@@ -589,6 +589,54 @@ def pasopel_main(args):
         print(json.dumps(_zufulix_arm(args, name, time_arm, hbm, tf, peak_kind)), flush=True)
 
 
+PN_SIZES = {
+    # width; heads / key-value heads / head sizes of the delta-rule and attention layers, convolution taps; matrix memory heads / head
+    # sizes; dense ff; vocab.  Width, depth, head counts, head sizes, taps, dense ff and vocabulary are those of DG_SIZES
+    "w1024": dict(width=1024, heads=8, kv_heads=2, dim=128, vdim=128, conv=4, mm_heads=4, mm_dim=128, mm_vdim=128, dense_ff=2816, vocab=32768),
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, conv=4, mm_heads=8, mm_dim=128, mm_vdim=128, dense_ff=5632, vocab=32768),
+}
+
+
+def panupel_main(args):
+    """Prefill and decode throughput of the Panupel family (delta rule, attention beside a matrix memory, delta rule, attention beside
+    a matrix memory, all with dense feed-forwards; the two middle layers form a loop that runs once) beside the closest existing
+    family, a Degavik stack of equal width, depth, head counts, head sizes and vocabulary."""
+    from ai00_server_b200 import runtime, synth
+    peaks, peak_kind = read_peaks()
+    hbm, tf = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    B, ctx = args.batch, args.context
+    time_arm = _family_timer(args, np.random.default_rng(7))
+    L = synth.panupel_layer
+    for name in args.kx_sizes.split(","):
+        z = PN_SIZES[name]
+        W, V, H, G, dk, dv, ff = z["width"], z["vocab"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["dense_ff"]
+        Hm, mk, mv = z["mm_heads"], z["mm_dim"], z["mm_vdim"]
+        hd = dict(heads=H, kv_heads=G, dim=dk, vdim=dv, ff=ff)
+        par = dict(base=5e5, scaling=(8.0, 1.0, 4.0, 8192), mm_heads=Hm, mm_dim=mk, mm_vdim=mv, **hd)
+        layers = [L("delta", conv=z["conv"], **hd), L("parallel", **par), L("delta", conv=z["conv"], **hd), L("parallel", **par)]
+        cfg, st, _ = synth.make_panupel(layers, width=W, vocab=V, seed=1, loop=(1, 3, 1), arrays=False)
+        # algorithmic work: weights one token touches (a decode step streams the same ones), recurrent states read and written, cache
+        # rows of the whole context in the two attention layers
+        mix_d = 2 * G * dk * W + 2 * H * dv * W + 2 * H * W + W * H * dv
+        mix_p = H * dk * W + G * (dk + dv) * W + H * W + W * H * dv + Hm * (2 * mk + 2 * mv + 2) * W + W * Hm * mv
+        active = 2 * mix_d + 2 * mix_p + 4 * 3 * W * ff + 2 * W * W + V * W
+        state_bytes = 2 * B * (H * dk * dv + Hm * mk * mv) * 4 * 2
+        step_bytes = 2 * active + state_bytes + 2 * B * ctx * G * (dk + dv) * 4
+        attn_flops_tok = 2 * 2 * H * (dk + dv) * ctx / 2 + 2 * 2 * 2 * (H * dk * dv + Hm * mk * mv)     # scores + values, state update + read-out
+        m = runtime.Model(st, max_batch=B, token_chunk_size=512, config=cfg, kv_tokens=B * (ctx + args.warmup + args.steps + 8))
+        r = time_arm(m, V, m.state.reset)
+        m.close()
+        r.update({"family": "panupel", "size": name, "batch": B, "context": ctx, "params_active_per_token": int(active),
+                  "decode_algorithmic_bytes_per_step": int(step_bytes),
+                  "decode_frac_of_hbm_peak": step_bytes / (r["decode_ms_per_step"] * 1e-3) / (hbm * 1e9),
+                  "prefill_tflops": (2 * active + attn_flops_tok) * r["prefill_tokens_per_s"] / 1e12,
+                  "prefill_frac_of_bf16_peak": (2 * active + attn_flops_tok) * r["prefill_tokens_per_s"] / 1e12 / tf,
+                  "peaks": peak_kind, "dtype": "bf16", "data": "synthetic"})
+        print(json.dumps(r), flush=True)
+        del st
+        print(json.dumps(_degavik_arm(args, name, time_arm, hbm, tf, peak_kind)), flush=True)
+
+
 def main():
     global PRESET, BATCH
     ap = argparse.ArgumentParser()
@@ -607,14 +655,14 @@ def main():
     ap.add_argument("--quant-layers", type=int, default=-1, help="the reference's `quant`: first N layers (default: all)")
     ap.add_argument("--seqs", type=int, default=256)
     ap.add_argument("--seq-len", type=int, default=512)
-    ap.add_argument("--family", default="rwkv", choices=["rwkv", "kemirax", "degavik", "zufulix", "pasopel"],
-                    help="kemirax / degavik / zufulix / pasopel: prefill and decode throughput of that family at layer sizes of a real model (random "
+    ap.add_argument("--family", default="rwkv", choices=["rwkv", "kemirax", "degavik", "zufulix", "pasopel", "panupel"],
+                    help="kemirax / degavik / zufulix / pasopel / panupel: prefill and decode throughput of that family at layer sizes of a real model (random "
                          "weights), beside the closest existing family at equal width and depth (RWKV-7 for kemirax, Kemirax for degavik, "
-                         "Degavik for zufulix, Zufulix for pasopel); one "
+                         "Degavik for zufulix, Zufulix for pasopel, Degavik for panupel); one "
                          "JSON line per arm (not the headline workload)")
-    ap.add_argument("--kx-sizes", default="w1024,w2048", help="--family kemirax / degavik / zufulix: comma-separated size names")
+    ap.add_argument("--kx-sizes", default="w1024,w2048", help="--family other than rwkv: comma-separated size names")
     ap.add_argument("--context", type=int, default=1024,
-                    help="--family kemirax / degavik / zufulix: tokens each sequence holds before the timed decode steps")
+                    help="--family other than rwkv: tokens each sequence holds before the timed decode steps")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     if args.family == "kemirax":
@@ -625,6 +673,8 @@ def main():
         return zufulix_main(args)
     if args.family == "pasopel":
         return pasopel_main(args)
+    if args.family == "panupel":
+        return panupel_main(args)
     PRESET, BATCH = args.preset, args.batch
     METRIC = metric_name(PRESET, BATCH)
     if args.quant != "none":
