@@ -165,7 +165,7 @@ void b200rwkv_engine::dg_load(const StFile& st, KxSizes& z) {
             while (l.wa_gt > 1 && window_attn_smem(qb, l.c.heads, l.c.dim, l.c.vdim, l.wa_gt) > 160 * 1024) l.wa_gt = (l.wa_gt + 1) / 2;
         }
     CK(cudaFuncSetAttribute(retention_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    CK(cudaFuncSetAttribute(delta_scan_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    CK(cudaFuncSetAttribute(delta_scan_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SCAN_SMEM));
     CK(cudaFuncSetAttribute(window_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     // the largest cluster the attention launch may ask for: what the device can co-schedule at this layer's shared memory
     m.max_split = 8;
@@ -237,7 +237,7 @@ void b200rwkv_engine::dg_enqueue_layer(cudaStream_t s, KxLayer& l, int rows, int
         const ScanShape sh = scan_shape(dk, dv, 3, decode);
         DeltaScanParams dp{m.cv, m.cv + G_ * dk, m.cv + 2 * G_ * dk, C_, m.z, H_ * dk, m.pr + C_, PN, l.a_log, l.rec_state, H_, G_, dk, dv,
                            1.f / sqrtf((float)dk), 1e-6f, sh, {m.vout, H_ * dv, nullptr, m.gl, H_ * dv, l.norm_w, 0, H_, dv, m.cfg.eps, 1.f, 0, mv}};
-        launch_k(delta_scan_kernel<true>, dim3(H_ * sh.ncta, nslot_grid), dim3(sh.threads), sh.smem_floats() * 4, dp, KC_WKV, s, prof);
+        launch_k(decode ? delta_scan_kernel<true, true> : delta_scan_kernel<true, false>, dim3(H_ * sh.ncta, nslot_grid), dim3(sh.threads), sh.smem_floats() * 4, dp, KC_WKV, s, prof);
         if (sh.ncta > 1) launch_k(head_norm_kernel, dim3(rows, cdiv(H_, 4)), dim3(128), 0, dp.norm, KC_LN, s, prof);
     } else {
         AttnPrepParams ap{m.pr, m.pr + H_ * dk, m.pr + H_ * dk + G_ * dk, PN, m.q, H_ * dk, l.cache, m.d_table, m.npages, m.page, l.qn_w, l.kn_w,

@@ -104,8 +104,8 @@ struct DeltaScanParams {
     HeadNormParams norm;                          // norm.x: raw read-outs, normed and gated in place
 };
 
-template <bool CHANNEL>
-__global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(const DeltaScanParams p) {
+template <bool CHANNEL, bool STEP>
+__global__ void __launch_bounds__(SCAN_THREADS, STEP ? 2 : 1) delta_scan_kernel(const DeltaScanParams p) {
     const ScanShape& sh = p.s;
     const int h = blockIdx.x / sh.ncta, cb = blockIdx.x % sh.ncta, si = blockIdx.y;
     const MetaView& meta = p.norm.meta;
@@ -120,8 +120,16 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(const DeltaSca
     float4* sscal = reinterpret_cast<float4*>(sbuf + (size_t)sh.nbuf * sh.tc * tokf);      // [tc] (decay, beta, 1 / |k|, q_scale / |q|)
     float* sraw = reinterpret_cast<float*>(sscal + sh.tc);        // [nbuf][tc][2] decay and write-strength logits
     float* rec = p.state + ((size_t)slot * p.H + h) * ((size_t)ks * sh.rt * dv);
+    __shared__ float red[SCAN_THREADS / 32];
+    const bool mine = part == 0 && col < ncol;    // this thread writes the column's read-outs
     float s[SCAN_R];
     scan_load_state(sh, rec, dv, j, part, s);
+    const float a_log = p.a_log[h];
+    float g_j = 0.f, w_j = 0.f, o_last = 0.f;     // STEP: gate and weight of the column, asked for early
+    if (STEP && mine && sh.ncta == 1) {
+        g_j = p.norm.gate[(size_t)t0 * p.norm.ldg + (size_t)h * dv + j];
+        w_j = p.norm.w[(size_t)h * p.norm.w_hstride + j];
+    }
     for (int e = x; e < sh.nbuf * sh.tc * tokf; e += blockDim.x) sbuf[e] = 0.f;
     __syncthreads();
     auto stage = [&](int c) {
@@ -138,14 +146,14 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(const DeltaSca
         }
         asm volatile("cp.async.commit_group;\n" ::: "memory");
     };
-    const float rate = expf(p.a_log[h]);
-    const int nc = (nt + sh.tc - 1) / sh.tc;
+    const int nc = STEP ? 1 : (nt + sh.tc - 1) / sh.tc;
     stage(0);
+    const float rate = expf(a_log);
     for (int c = 0; c < nc; ++c) {
-        const int n = min(sh.tc, nt - c * sh.tc);
+        const int n = STEP ? 1 : min(sh.tc, nt - c * sh.tc);
         float* buf = sbuf + (size_t)(c % sh.nbuf) * sh.tc * tokf;
         const float* raw = sraw + (size_t)(c % sh.nbuf) * sh.tc * 2;
-        if (sh.nbuf > 1 && c + 1 < nc) {
+        if (!STEP && c + 1 < nc) {
             stage(c + 1);                          // into the buffer that group c - 1 used: everyone left it at the barrier below
             asm volatile("cp.async.wait_group 1;\n" ::: "memory");
         } else {
@@ -194,6 +202,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(const DeltaSca
             }
             const float d = scan_part_sum((d0 + d1) + (d2 + d3), ks);
             const float u = sc.y * (vj - d * sc.z) * sc.z;         // u / |k|: the write is (k / |k|) u^T
+            if (STEP) asm volatile("" ::: "memory");     // read the key again below instead of keeping it: 64 registers, two CTAs per SM
             float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
 #pragma unroll
             for (int r = 0; r < SCAN_R; r += 4) {
@@ -202,13 +211,26 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(const DeltaSca
                 o0 = fmaf(s[r], q4.x, o0); o1 = fmaf(s[r + 1], q4.y, o1); o2 = fmaf(s[r + 2], q4.z, o2); o3 = fmaf(s[r + 3], q4.w, o3);
             }
             const float o = scan_part_sum((o0 + o1) + (o2 + o3), ks) * sc.w;
-            if (part == 0 && col < ncol) orow[(size_t)t * p.norm.ldx] = o;
+            if (STEP && sh.ncta == 1) o_last = o;
+            else if (mine) orow[(size_t)t * p.norm.ldx] = o;
         }
-        __syncthreads();
+        if (!STEP) __syncthreads();
     }
     scan_store_state(sh, rec, dv, j, part, s);
-    if (sh.ncta == 1)
+    if constexpr (STEP) {
+        if (sh.ncta == 1) {                        // the CTA holds the head: norm and gate from registers
+            float ss = mine ? o_last * o_last : 0.f;
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            if (lane == 0) red[warp] = ss;
+            __syncthreads();
+            ss = 0.f;
+            for (int w = 0; w < nw; ++w) ss += red[w];
+            if (mine) p.norm.x[(size_t)t0 * p.norm.ldx + (size_t)h * dv + j] = head_norm_value(p.norm, o_last, 1.f, ss, w_j, g_j);
+        }
+    } else if (sh.ncta == 1) {
         for (int t = warp; t < nt; t += nw) head_norm_row(p.norm, t0 + t, h, lane);
+    }
 }
 
 }  // namespace b200

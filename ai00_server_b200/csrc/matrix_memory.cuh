@@ -35,7 +35,8 @@ struct MatrixMemoryParams {
 
 constexpr int MM_MAX_N = SCAN_MAX_DK / SCAN_THREADS_PROMPT;      // normaliser entries per thread
 
-__global__ void __launch_bounds__(SCAN_THREADS) matrix_memory_kernel(const MatrixMemoryParams p) {
+template <bool STEP>
+__global__ void __launch_bounds__(SCAN_THREADS, STEP ? 2 : 1) matrix_memory_kernel(const MatrixMemoryParams p) {
     const ScanShape& sh = p.s;
     const int h = blockIdx.x / sh.ncta, cb = blockIdx.x % sh.ncta, si = blockIdx.y;
     const MetaView& meta = p.norm.meta;
@@ -54,15 +55,24 @@ __global__ void __launch_bounds__(SCAN_THREADS) matrix_memory_kernel(const Matri
     float* rec = p.state + hs * ((size_t)ks * sh.rt * dv);
     float* gn = p.n + hs * dk;
     float* gm = p.m + hs * dv + cb * sh.cols;
+    __shared__ float red[SCAN_THREADS / 32];
+    const bool mine = part == 0 && col < ncol;     // this thread writes the column's read-outs
     float s[SCAN_R];
     scan_load_state(sh, rec, dv, j, part, s);
-    float n[MM_MAX_N];
-    int noff[MM_MAX_N];                            // staged place of this thread's entries of the key dimension
+    float g_j = 0.f, w_j = 0.f, o_last = 0.f;      // STEP: gate and weight of the column, asked for early
+    if (STEP && mine && sh.ncta == 1) {
+        g_j = p.norm.gate[(size_t)t0 * p.norm.ldg + (size_t)h * dv + j];
+        w_j = p.norm.w[(size_t)h * p.norm.w_hstride + j];
+    }
+    constexpr int NE = STEP ? 1 : MM_MAX_N;        // STEP: the first entry is asked for early, further ones are met in memory
+    float n[NE];
+    int noff[NE];                                  // staged place of this thread's entries of the key dimension
+    auto place = [&](int i) { return i / sh.rt * SCAN_ROW + i % sh.rt; };
 #pragma unroll
-    for (int e = 0; e < MM_MAX_N; ++e) {
+    for (int e = 0; e < NE; ++e) {
         const int i = e * nthr + x;
-        n[e] = 0.f; noff[e] = SCAN_R;   // place 32 of part 0 is padding: always zero
-        if (cb == 0 && i < dk) { n[e] = gn[i]; noff[e] = i / sh.rt * SCAN_ROW + i % sh.rt; }
+        n[e] = 0.f; noff[e] = SCAN_R;              // place 32 of part 0 is padding: always zero
+        if (cb == 0 && i < dk) { n[e] = gn[i]; noff[e] = place(i); }
     }
     float m_run = gm[0];                           // meaningful in warp 0
     for (int e = x; e < sh.nbuf * sh.tc * tokf; e += nthr) sbuf[e] = 0.f;
@@ -80,13 +90,13 @@ __global__ void __launch_bounds__(SCAN_THREADS) matrix_memory_kernel(const Matri
         }
         asm volatile("cp.async.commit_group;\n" ::: "memory");
     };
-    const int nc = (nt + sh.tc - 1) / sh.tc;
+    const int nc = STEP ? 1 : (nt + sh.tc - 1) / sh.tc;
     stage(0);
     for (int c = 0; c < nc; ++c) {
-        const int cnt = min(sh.tc, nt - c * sh.tc);
+        const int cnt = STEP ? 1 : min(sh.tc, nt - c * sh.tc);
         float* buf = sbuf + (size_t)(c % sh.nbuf) * sh.tc * tokf;
         const float* raw = sraw + (size_t)(c % sh.nbuf) * sh.tc * 2;
-        if (sh.nbuf > 1 && c + 1 < nc) {
+        if (!STEP && c + 1 < nc) {
             stage(c + 1);                          // into the buffer that group c - 1 used: everyone left it at the barrier below
             asm volatile("cp.async.wait_group 1;\n" ::: "memory");
         } else {
@@ -123,35 +133,56 @@ __global__ void __launch_bounds__(SCAN_THREADS) matrix_memory_kernel(const Matri
                 o0 = fmaf(s[r], q4.x, o0); o1 = fmaf(s[r + 1], q4.y, o1); o2 = fmaf(s[r + 2], q4.z, o2); o3 = fmaf(s[r + 3], q4.w, o3);
             }
             const float o = scan_part_sum((o0 + o1) + (o2 + o3), ks);
-            if (part == 0 && col < ncol) orow[(size_t)t * p.norm.ldx] = o;
+            if (STEP && sh.ncta == 1) o_last = o;
+            else if (mine) orow[(size_t)t * p.norm.ldx] = o;
             if (cb == 0) {                         // the normaliser and its product with the query
                 float nq = 0.f;
 #pragma unroll
-                for (int e = 0; e < MM_MAX_N; ++e) {
+                for (int e = 0; e < NE; ++e) {
                     if (e * nthr >= dk) break;     // the same for all threads
                     n[e] = fmaf(sc.y, row[noff[e]], sc.x * n[e]);
                     nq = fmaf(n[e], row[krow + noff[e]], nq);
                 }
+                if (STEP)
+                    for (int i = nthr + x; i < dk; i += nthr) {
+                        const float v = fmaf(sc.y, row[place(i)], sc.x * gn[i]);
+                        gn[i] = v;
+                        nq = fmaf(v, row[krow + place(i)], nq);
+                    }
 #pragma unroll
                 for (int o2_ = 16; o2_ > 0; o2_ >>= 1) nq += __shfl_xor_sync(0xffffffffu, nq, o2_);
                 if (lane == 0) snq[t * nw + warp] = nq;
             }
         }
+        if constexpr (STEP) {
+            float ss = mine ? o_last * o_last : 0.f;
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            if (lane == 0) red[warp] = ss;
+        }
         __syncthreads();
-        if (cb == 0 && x < cnt) {
+        if (STEP ? cb == 0 : (cb == 0 && x < cnt)) {
+            const int u = STEP ? 0 : x;
             float nq = 0.f;
-            for (int w = 0; w < nw; ++w) nq += snq[x * nw + w];
-            p.fac[(size_t)(t0 + c * sh.tc + x) * p.H + h] = p.q_scale / (fmaxf(fabsf(nq * p.q_scale), sscal[x].z) + p.den_eps);
+            for (int w = 0; w < nw; ++w) nq += snq[u * nw + w];
+            const float fac = p.q_scale / (fmaxf(fabsf(nq * p.q_scale), sscal[u].z) + p.den_eps);
+            if (STEP && sh.ncta == 1) {            // the CTA holds the head: norm and gate from registers
+                float ss = 0.f;
+                for (int w = 0; w < nw; ++w) ss += red[w];
+                if (mine) p.norm.x[(size_t)t0 * p.norm.ldx + (size_t)h * dv + j] = head_norm_value(p.norm, o_last, fac, ss, w_j, g_j);
+            } else if (!STEP || x == 0) {
+                p.fac[(size_t)(t0 + c * sh.tc + u) * p.H + h] = fac;
+            }
         }
     }
     scan_store_state(sh, rec, dv, j, part, s);
     if (cb == 0)
 #pragma unroll
-        for (int e = 0; e < MM_MAX_N; ++e)
+        for (int e = 0; e < NE; ++e)
             if (e * nthr + x < dk) gn[e * nthr + x] = n[e];
     if (warp == 0)
         for (int i = lane; i < ncol; i += 32) gm[i] = m_run;
-    if (sh.ncta == 1) {
+    if (!STEP && sh.ncta == 1) {
         __syncthreads();                           // the factors of all tokens are written
         for (int t = warp; t < nt; t += nw) head_norm_row(p.norm, t0 + t, h, lane);
     }

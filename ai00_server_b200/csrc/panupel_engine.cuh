@@ -135,8 +135,8 @@ void b200rwkv_engine::pn_load(const StFile& st, KxSizes& z) {
         if (c.has_mlp) z.n_ys = std::max(z.n_ys, (size_t)c.ff);
     }
     sa_plan_model(m);
-    CK(cudaFuncSetAttribute(delta_scan_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    CK(cudaFuncSetAttribute(matrix_memory_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    CK(cudaFuncSetAttribute(delta_scan_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SCAN_SMEM));
+    CK(cudaFuncSetAttribute(matrix_memory_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SCAN_SMEM));
     REQUIRE((size_t)W * 4 <= 200 * 1024, B200RWKV_ERR_UNSUPPORTED, "width too large for the norm kernel");
     CK(cudaFuncSetAttribute(pre_norm_kernel<NORM_THREADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     CK(cudaFuncSetAttribute(pre_norm_kernel<PRE_NORM_THREADS_FEW_ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
@@ -192,7 +192,7 @@ void b200rwkv_engine::pn_enqueue_layers(cudaStream_t s, int rows, int nslot_grid
                 MatrixMemoryParams mp{m.pr + r.mq, m.pr + r.mk, m.pr + r.mv, PN, m.pr + r.mi, m.pr + r.mf, l.mm_state, l.mm_n, l.mm_m, m.z, Hm, mk, mvd,
                                       c.mm_cap, 1.f / sqrtf((float)mk), 1e-6f, sh,
                                       {m.vout + H_ * dv, KO, m.z, m.pr + r.mg, PN, l.mm_norm_w, mvd, Hm, mvd, eps, c.mm_mul, 0, mv}};
-                launch_k(matrix_memory_kernel, dim3(Hm * sh.ncta, nslot_grid), dim3(sh.threads), sh.smem_floats() * 4, mp, KC_WKV, s2, prof);
+                launch_k(decode ? matrix_memory_kernel<true> : matrix_memory_kernel<false>, dim3(Hm * sh.ncta, nslot_grid), dim3(sh.threads), sh.smem_floats() * 4, mp, KC_WKV, s2, prof);
                 if (sh.ncta > 1) launch_k(head_norm_kernel, dim3(rows, cdiv(Hm, 4)), dim3(128), 0, mp.norm, KC_LN, s2, prof);
             }
             RotPrepParams rp{m.pr + r.q, m.pr + r.k, m.pr + r.v, PN, m.q, H_ * dk, l.cache, m.d_table, m.npages, m.page, l.qn_w, l.kn_w, l.freq_d,
@@ -219,7 +219,7 @@ void b200rwkv_engine::pn_enqueue_layers(cudaStream_t s, int rows, int nslot_grid
             const ScanShape sh = scan_shape(dk, dv, 2, decode);
             DeltaScanParams dp{m.cv, m.cv + G_ * dk, m.cv + 2 * G_ * dk, ldc, m.pr + r.a, PN, m.pr + r.b, PN, l.a_log, l.rec_state, H_, G_, dk, dv,
                                1.f / sqrtf((float)dk), 1e-6f, sh, {m.vout, KO, nullptr, m.pr + r.g, PN, l.norm_w, 0, H_, dv, eps, 1.f, 1, mv}};
-            launch_k(delta_scan_kernel<false>, dim3(H_ * sh.ncta, nslot_grid), dim3(sh.threads), sh.smem_floats() * 4, dp, KC_WKV, s, prof);
+            launch_k(decode ? delta_scan_kernel<false, true> : delta_scan_kernel<false, false>, dim3(H_ * sh.ncta, nslot_grid), dim3(sh.threads), sh.smem_floats() * 4, dp, KC_WKV, s, prof);
             if (sh.ncta > 1) launch_k(head_norm_kernel, dim3(rows, cdiv(H_, 4)), dim3(128), 0, dp.norm, KC_LN, s, prof);
         }
         kx_lin(s, prof, lin(m.vout, KO, l.o, m.y, W, W, KO), rows, 1);

@@ -12,7 +12,8 @@
 // i % rt of part i / rt; entries past dk are zero and stay zero.
 //
 // The raw read-outs go to the output rows; the root-mean-square norm over a head, its weight, a gate and a constant are applied in
-// place afterwards: by the same CTA where it holds the whole head, by head_norm_kernel otherwise.
+// place afterwards: by the same CTA where it holds the whole head, by head_norm_kernel otherwise.  In steps of one token per sequence
+// (kernel template STEP) a CTA that holds the whole head keeps the read-outs in registers and finishes them on the spot.
 #pragma once
 #include <cuda_runtime.h>
 #include "common.cuh"
@@ -25,6 +26,7 @@ constexpr int SCAN_ROW = SCAN_R + 4;               // staged floats per part: ei
 constexpr int SCAN_MAX_DK = 32 * SCAN_R;
 constexpr int SCAN_THREADS = 512;                  // most threads per CTA (a whole head at once: steps of one token per sequence)
 constexpr int SCAN_THREADS_PROMPT = 128;
+constexpr int SCAN_SMEM = 64 * 1024;               // most shared memory of a launch
 
 struct ScanShape {
     int ks, lks, rt;                               // lanes per column (a power of two and its logarithm), entries per lane (a multiple of 4)
@@ -59,7 +61,7 @@ __host__ inline ScanShape scan_shape(int dk, int dv, int rows, bool decode) {
     s.ncta = (dv + s.cols - 1) / s.cols;
     s.nbuf = decode ? 1 : 2;
     s.tc = decode ? 1 : 16;
-    while (s.tc > 1 && s.smem_floats() * sizeof(float) > 64 * 1024) s.tc /= 2;
+    while (s.tc > 1 && s.smem_floats() * sizeof(float) > SCAN_SMEM) s.tc /= 2;
     return s;
 }
 
@@ -141,6 +143,12 @@ __device__ __forceinline__ void head_norm_row(const HeadNormParams& p, int t, in
         const float gl = g[j], a = lin_sigmoid(gl);
         x[j] = x[j] * f * r * w[j] * (p.silu ? gl * a : a) * p.mul;
     }
+}
+
+// the same for one entry o of a read-out whose sum of squares is known
+__device__ __forceinline__ float head_norm_value(const HeadNormParams& p, float o, float f, float ss, float w, float gate) {
+    const float a = lin_sigmoid(gate);
+    return o * f / sqrtf(f * f * ss / (float)p.dv + p.eps) * w * (p.silu ? gate * a : a) * p.mul;
 }
 
 __global__ void __launch_bounds__(128) head_norm_kernel(const HeadNormParams p) {

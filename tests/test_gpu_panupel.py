@@ -29,7 +29,8 @@ def row_errs(got, want):
 
 def exact(got, want):
     e = row_errs(got, want)
-    assert len(e) == len(want) and e.max() <= TIGHT and np.median(e) <= TYPICAL, (e.argmax(), e.max(), np.median(e))
+    assert len(e) == len(want) and e.max() <= TIGHT, (e.argmax(), e.max())
+    assert len(e) < 20 or np.median(e) <= TYPICAL, np.median(e)
 
 
 class Bundle:
