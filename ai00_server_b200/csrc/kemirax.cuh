@@ -320,7 +320,7 @@ struct KxLayer {
     float *qn_w = nullptr, *kn_w = nullptr, *talk = nullptr, *temp = nullptr;   // windowed attention
     double* freq_d = nullptr;                                    // rotary frequencies in double (retention, windowed attention)
     int wa_gt = 1;                                               // key / value heads per tile load of the attention kernel
-    float* rec_state = nullptr;                                  // retention / delta rule: [S][H][dk][dv]
+    float* rec_state = nullptr;                                  // retention: [S][H][dk][dv]; delta rule: [S][H] state records (state_scan.cuh)
     int cache_D = 0;                                             // floats per cached token when the layer owns a pool
     // Zufulix: layer norms with bias, stream coefficients of the two sublayers, projection biases, distance-bias table
     float *norm1_b = nullptr, *norm2_b = nullptr;
