@@ -47,6 +47,7 @@ ARCH_DEGAVIK = 101
 ARCH_ZUFULIX = 102
 ARCH_PASOPEL = 103
 ARCH_PANUPEL = 104
+ARCH_FUFIPEL = 105
 
 
 class B200Error(RuntimeError):

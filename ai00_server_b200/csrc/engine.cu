@@ -296,11 +296,13 @@ static b200rwkv_info derive_info(const StFile& st) {
         const StTensor& e = *st.find("embed");
         // Kemirax norms are one gain; Degavik norms are weight vectors (and a layer may have no tensors of its own); Zufulix
         // norms have a bias and the embedding table doubles as the output matrix; Pasopel has vector norms without a bias and
-        // no separate output matrix either; Panupel layers have a second norm around every mixer
+        // no separate output matrix either; Panupel layers have a second norm around every mixer; Fufipel is like Pasopel there, with
+        // a distance-bias table or a norm on one half of a mixer in its first layer
         o.version = st.find("final.norm.b") ? B200RWKV_ARCH_ZUFULIX
                     : st.find("final.norm")->numel() == 1 ? B200RWKV_ARCH_KEMIRAX
                     : st.find("l0.norm1b") ? B200RWKV_ARCH_PANUPEL
-                    : (st.find("head") ? B200RWKV_ARCH_DEGAVIK : B200RWKV_ARCH_PASOPEL);
+                    : st.find("head") ? B200RWKV_ARCH_DEGAVIK
+                    : (st.find("l0.mix.rel") || st.find("l0.mix.left.out") ? B200RWKV_ARCH_FUFIPEL : B200RWKV_ARCH_PASOPEL);
         o.num_vocab = (int)StFile::dim(e, 0, "embed", 2);
         o.num_emb = (int)StFile::dim(e, 1, "embed", 2);
         if (o.version != B200RWKV_ARCH_DEGAVIK) {
@@ -426,6 +428,7 @@ struct Snapshot { float* buf = nullptr; float* logits = nullptr; size_t bytes = 
 #include "zufulix.cuh"
 #include "pasopel.cuh"
 #include "panupel.cuh"
+#include "fufipel.cuh"
 
 using namespace b200;
 
@@ -543,10 +546,14 @@ struct b200rwkv_engine {
     void ps_repool(int slot, int n);
     void pn_load(const StFile& st, KxSizes& z);                   // Panupel family (panupel_engine.cuh)
     void pn_enqueue_layers(cudaStream_t s, int rows, int nslot_grid, bool decode, int nsplit, Profiler* prof);
+    void ff_load(const StFile& st, KxSizes& z);                   // Fufipel family (fufipel_engine.cuh)
+    void ff_enqueue_layers(cudaStream_t s, int rows, int nslot_grid, bool decode, int nsplit, Profiler* prof);
     __nv_bfloat16* kx_up16(const std::vector<uint16_t>& v);
     float* kx_up32(const std::vector<float>& v);
     void kx_lin(cudaStream_t s, Profiler* prof, LinParams p, int rows, int groups, bool force_exact = false);
     void kx_short_conv(cudaStream_t s, Profiler* prof, const ShortConvParams& cp, int rows, int nslot_grid, bool decode);
+    void kx_gla(cudaStream_t s, Profiler* prof, const KxLayer& l, int H_, int dk, int dv, const float* q, const float* k, const float* v,
+                const float* gate, int ld, float* out, int ldo, int rows, int nslot_grid, bool decode);
     void kx_enqueue_step(cudaStream_t s, int rows, int rrows, bool decode, int nsplit, Profiler* prof);
     void kx_fill_step(int* hm, const std::vector<int>& slots, const std::vector<int>& counts, bool* decode, int* nsplit);
     void kx_run_step(int T, int R, bool decode, int nsplit);
@@ -1855,6 +1862,7 @@ void b200rwkv_engine::state_xform(int slot, bool import, float* snap) {
 #include "sink_attn_plan.cuh"
 #include "pasopel_engine.cuh"
 #include "panupel_engine.cuh"
+#include "fufipel_engine.cuh"
 
 // =========================================================================================
 // in-process tensor-parallel group

@@ -110,8 +110,10 @@ struct RotCfg {
     bool banded = false; double low = 0, high = 0;                                     // bands of wavelengths (kx_rot_freqs), with factor and original
 };
 
-enum KxMixer { KX_LATENT = 0, KX_GLA = 1, KX_RETENTION = 2, KX_DELTA = 3, KX_WINDOW = 4, KX_BIASED = 5, KX_SINK = 6, KX_PARALLEL = 7 };
-enum KxFamily { KX_FAMILY_KEMIRAX = 0, KX_FAMILY_DEGAVIK = 1, KX_FAMILY_ZUFULIX = 2, KX_FAMILY_PASOPEL = 3, KX_FAMILY_PANUPEL = 4 };
+enum KxMixer { KX_LATENT = 0, KX_GLA = 1, KX_RETENTION = 2, KX_DELTA = 3, KX_WINDOW = 4, KX_BIASED = 5, KX_SINK = 6, KX_PARALLEL = 7,
+               KX_BIAS_WINDOW = 8, KX_CHUNK_GLA = 9 };
+enum KxFamily { KX_FAMILY_KEMIRAX = 0, KX_FAMILY_DEGAVIK = 1, KX_FAMILY_ZUFULIX = 2, KX_FAMILY_PASOPEL = 3, KX_FAMILY_PANUPEL = 4,
+                KX_FAMILY_FUFIPEL = 5 };
 
 struct KxLayerCfg {
     int mixer = KX_LATENT;
@@ -138,6 +140,9 @@ struct KxLayerCfg {
     int mm_heads = 0, mm_dim = 0, mm_vdim = 0;                   // matrix memory
     float mm_cap = 0.f;                                          // its gates' pre-activations are squashed by cap * tanh(z / cap)
     float attn_mul = 1.f, mm_mul = 1.f;                          // factors on the two sides' outputs
+    // Fufipel (fufipel.cuh): windowed attention with a distance bias; attention inside chunks of `chunk` tokens beside gated linear
+    // attention (its heads and sizes: mm_heads, mm_dim, mm_vdim)
+    int chunk = 0;
     int rot_dim = 0, kv_rank = 0, q_rank = 0, kv_from = -1;     // latent attention
     float scale = 1.f;
     RotCfg rot;
@@ -158,6 +163,8 @@ struct KxConfig {
     float embed_scale = 1.f;                                     // factor on the embedding row
     float logit_cap = 0.f;                                       // logits <- cap * tanh(logits / cap) (0: none)
     float residual_mul = 1.f;                                    // factor on every sublayer's contribution to the residual
+    int pair_buckets = 0, pair_mul_prev = 0, pair_mul_cur = 0;   // embedding of (previous token, token) pairs (rmsnorm.cuh); 0: none
+    float logit_scale = 1.f;                                     // factor on the logits
     bool has_loop = false;                                       // a run of layers is executed several times (`layers` lists every run)
     std::vector<KxLayerCfg> layers;
 };
@@ -166,6 +173,7 @@ static KxConfig dg_parse_config(const JVal& root);
 static KxConfig zf_parse_config(const JVal& root);
 static KxConfig ps_parse_config(const JVal& root);
 static KxConfig pn_parse_config(const JVal& root);
+static KxConfig ff_parse_config(const JVal& root);
 
 // model registry of the families that come with a config.json: `architecture` names the design
 static KxConfig kx_parse_config(const char* json, size_t n) {
@@ -177,6 +185,7 @@ static KxConfig kx_parse_config(const char* json, size_t n) {
     if (arch == "Zufulix") return zf_parse_config(root);
     if (arch == "Pasopel") return ps_parse_config(root);
     if (arch == "Panupel") return pn_parse_config(root);
+    if (arch == "Fufipel") return ff_parse_config(root);
     REQUIRE(arch == "Kemirax", B200RWKV_ERR_UNSUPPORTED, "config: unknown architecture '" + arch + "'");
     KxConfig c;
     c.vocab = root.integer("vocab");
@@ -227,25 +236,12 @@ static KxConfig kx_parse_config(const char* json, size_t n) {
 }
 
 // rotary frequency table with the long-context rescaling folded in (double arithmetic on the host, f32 table on the device)
+static std::vector<double> kx_rot_freqs(const RotCfg& r);
+static float kx_rot_mag(const RotCfg& r) { return r.scaled ? (float)(0.1 * std::log(r.factor) + 1.0) : 1.f; }      // factor on cosine and sine
 static void kx_rot_table(const RotCfg& r, std::vector<float>& freq, float& mag) {
-    const int half = r.dims / 2;
-    freq.resize(std::max(half, 1));
-    mag = 1.f;
-    int lo = 0, hi = 0;
-    if (r.scaled) {
-        auto turn_dim = [&](double turns) { return r.dims * std::log(r.original / (2.0 * M_PI * turns)) / (2.0 * std::log(r.base)); };
-        lo = std::max((int)std::floor(turn_dim(r.fast)), 0);
-        hi = std::min((int)std::ceil(turn_dim(r.slow)), r.dims - 1);
-        mag = (float)(0.1 * std::log(r.factor) + 1.0);
-    }
-    for (int i = 0; i < half; ++i) {
-        double f = std::pow(r.base, -2.0 * i / r.dims);
-        if (r.scaled) {
-            const double ramp = std::min(1.0, std::max(0.0, (i - lo) / std::max((double)(hi - lo), 0.001)));
-            f = f / r.factor * ramp + f * (1.0 - ramp);
-        }
-        freq[i] = (float)f;
-    }
+    const std::vector<double> f = kx_rot_freqs(r);
+    freq.assign(f.begin(), f.end());
+    mag = kx_rot_mag(r);
 }
 
 // `loop` of a config: layers start .. stop - 1 are executed `times` times in a row.  The layer runs go to c.layers in execution
@@ -274,12 +270,23 @@ static void kx_unroll_loop(const JVal& root, const std::vector<KxLayerCfg>& own,
     }
 }
 
-// rotary frequencies in double.  Banded: a pair whose wavelength is shorter than original / high keeps its frequency, one longer
+// rotary frequencies in double.  Scaled: a ramp over the pairs, from those that turn `fast` times over the original context (unchanged)
+// to those that turn `slow` times (`factor` times slower).  Banded: a pair whose wavelength is shorter than original / high keeps its frequency, one longer
 // than original / low turns `factor` times slower, and in between the two are blended linearly in original / wavelength
 static std::vector<double> kx_rot_freqs(const RotCfg& r) {
     std::vector<double> f(std::max(r.dims / 2, 1), 0.0);
+    double lo = 0, hi = 0;
+    if (r.scaled) {
+        auto turn_dim = [&](double turns) { return r.dims * std::log(r.original / (2.0 * M_PI * turns)) / (2.0 * std::log(r.base)); };
+        lo = std::max(std::floor(turn_dim(r.fast)), 0.0);
+        hi = std::min(std::ceil(turn_dim(r.slow)), r.dims - 1.0);
+    }
     for (int i = 0; i < r.dims / 2; ++i) {
         f[i] = std::pow(r.base, -2.0 * i / r.dims);
+        if (r.scaled) {
+            const double ramp = std::min(1.0, std::max(0.0, (i - lo) / std::max(hi - lo, 0.001)));
+            f[i] = f[i] / r.factor * ramp + f[i] * (1.0 - ramp);
+        }
         if (!r.banded) continue;
         const double wave = 2.0 * M_PI / f[i];
         if (wave < r.original / r.high) continue;
@@ -306,7 +313,7 @@ struct KxLayer {
     float* cache = nullptr;                       // [pages][page][rk + dr]; a borrowing layer points at the lender's pool
     // gla
     __nv_bfloat16 *proj = nullptr, *a2 = nullptr;               // proj = [q; k; v; g; a1] stacked
-    float *a2_b = nullptr, *norm_w = nullptr, *gla_state = nullptr;
+    float *a2_b = nullptr, *norm_w = nullptr, *gla_state = nullptr;      // gla_state: [S][H] state records (state_scan.cuh)
     int a_rank = 0, proj_n = 0;
     // feed-forward
     __nv_bfloat16 *router = nullptr, *gu = nullptr, *down = nullptr, *sh_gu = nullptr, *sh_down = nullptr, *sg = nullptr;
@@ -339,6 +346,8 @@ struct KxLayer {
     bool sa_reg = false;                                         // head sizes fit the register form of the attention kernel
     // Panupel: norms on the sublayers' outputs, matrix memory
     float *norm1b_w = nullptr, *norm2b_w = nullptr, *mm_norm_w = nullptr;
+    // Fufipel: norms on the two halves' outputs (norm1b_w, norm2b_w), output projection of the right half
+    __nv_bfloat16* o2 = nullptr;
     float *mm_state = nullptr, *mm_n = nullptr, *mm_m = nullptr;     // [S][H] x (state record of state_scan.cuh, dk floats, one float)
     // per-sequence memory of fixed size, in the order of the flat state record
     struct Block { float* base; size_t per_slot; };
@@ -384,6 +393,9 @@ struct SeqModel {
           *ds = nullptr, *hn = nullptr;
     int *sel = nullptr, *cnt = nullptr, *off = nullptr, *list = nullptr, *row_of = nullptr;
     float* lin_ws = nullptr; size_t lin_ws_floats = 0;
+    __nv_bfloat16* pairs = nullptr;               // [buckets + 1][W] embedding rows of token pairs
+    float* last_tok = nullptr;                    // [S] last token of every sequence (families with pair embeddings)
+    bool side_lin = false; float* lin_ws_side = nullptr;      // projections also run on the side stream: split-k sums of their own
     float* dbg_layers = nullptr;                  // [L][maxT][W] residual after every layer (bring-up aid; nullptr: off)
     int max_split = 16;
     int sa_ygroups = 1, sa_ygroups_decode = 1;    // head groups (grid rows) of the smallest windowed-attention launch of the model (prompt / decode shape)

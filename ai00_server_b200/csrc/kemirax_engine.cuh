@@ -136,8 +136,7 @@ void b200rwkv_engine::kx_load(const StFile& st, KxSizes& z) {
             m.max_D = std::max(m.max_D, D);
         } else {
             const int H_ = c.heads, dk = c.dim, dv = c.vdim;
-            REQUIRE(dv <= 1024, B200RWKV_ERR_UNSUPPORTED, "gla vdim must be <= 1024");
-            REQUIRE(gla_smem_bytes(dk, dv) <= 200 * 1024, B200RWKV_ERR_UNSUPPORTED, "gla head state too large for shared memory");
+            REQUIRE(dk <= SCAN_MAX_DK, B200RWKV_ERR_UNSUPPORTED, "gla: dim must be <= 1024");
             const StTensor* a1 = st.find(p + "mix.a1");
             REQUIRE(a1 && a1->shape.size() == 2, B200RWKV_ERR_INVALID, "missing tensor: " + p + "mix.a1");
             l.a_rank = (int)a1->shape[0];
@@ -152,8 +151,9 @@ void b200rwkv_engine::kx_load(const StFile& st, KxSizes& z) {
             l.a2_b = kx_up32(kx_host_f32(st, p + "mix.a2.b", (int64_t)H_ * dk));
             l.norm_w = kx_up32(kx_host_f32(st, p + "mix.norm", dv));
             l.o = kx_up16(kx_host_bf16(st, p + "mix.o", W, (int64_t)H_ * dv));
-            l.gla_state = (float*)dalloc((size_t)S * H_ * dk * dv * 4);
-            l.fixed.push_back({l.gla_state, (size_t)H_ * dk * dv});
+            const size_t per_slot = (size_t)H_ * scan_state_floats(dk, dv);
+            l.gla_state = (float*)dalloc((size_t)S * per_slot * 4);
+            l.fixed.push_back({l.gla_state, per_slot});
             z.n_pr = std::max(z.n_pr, (size_t)l.proj_n); z.n_z = std::max(z.n_z, (size_t)H_ * dk); z.n_vout = std::max(z.n_vout, (size_t)H_ * dv);
         }
         if (c.has_mlp) {
@@ -192,7 +192,8 @@ void b200rwkv_engine::kx_build(const StFile& st, const char* cfg_json, size_t cf
     m.W = m.cfg.width; m.V = m.cfg.vocab;
     const int W = m.W, nl = (int)m.cfg.layers.size();
     memset(&info, 0, sizeof(info));
-    info.version = m.cfg.family == KX_FAMILY_PANUPEL ? B200RWKV_ARCH_PANUPEL
+    info.version = m.cfg.family == KX_FAMILY_FUFIPEL ? B200RWKV_ARCH_FUFIPEL
+                   : m.cfg.family == KX_FAMILY_PANUPEL ? B200RWKV_ARCH_PANUPEL
                    : m.cfg.family == KX_FAMILY_PASOPEL ? B200RWKV_ARCH_PASOPEL
                    : m.cfg.family == KX_FAMILY_ZUFULIX ? B200RWKV_ARCH_ZUFULIX
                    : (m.cfg.family == KX_FAMILY_DEGAVIK ? B200RWKV_ARCH_DEGAVIK : B200RWKV_ARCH_KEMIRAX); info.num_layer = nl; info.num_emb = W; info.num_vocab = m.V;
@@ -227,7 +228,8 @@ void b200rwkv_engine::kx_build(const StFile& st, const char* cfg_json, size_t cf
     for (int i = m.npages - 1; i >= 0; --i) m.free_pages.push_back(i);
 
     KxSizes z;
-    if (m.cfg.family == KX_FAMILY_PANUPEL) pn_load(st, z);
+    if (m.cfg.family == KX_FAMILY_FUFIPEL) ff_load(st, z);
+    else if (m.cfg.family == KX_FAMILY_PANUPEL) pn_load(st, z);
     else if (m.cfg.family == KX_FAMILY_PASOPEL) ps_load(st, z);
     else if (m.cfg.family == KX_FAMILY_ZUFULIX) zf_load(st, z);
     else if (m.cfg.family == KX_FAMILY_DEGAVIK) dg_load(st, z);
@@ -245,6 +247,7 @@ void b200rwkv_engine::kx_build(const StFile& st, const char* cfg_json, size_t cf
     m.y = fa(T_ * W); m.cv = fa(T_ * z.n_cv); m.gl = fa(T_ * z.n_gl); m.vfirst = fa(T_ * z.n_vf);
     m.lin_ws_floats = (size_t)4 << 20;                   // split-k partial sums of one projection launch
     m.lin_ws = fa(m.lin_ws_floats);
+    if (m.side_lin) m.lin_ws_side = fa(m.lin_ws_floats);
     m.sel = (int*)dalloc(T_ * z.max_top * 4); m.row_of = (int*)dalloc(T_ * z.max_top * 4); m.list = (int*)dalloc(T_ * z.max_top * 4);
     m.cnt = (int*)dalloc((size_t)z.max_E * 4); m.off = (int*)dalloc((size_t)z.max_E * 4);
     d_hidden = fa(T_ * W);
@@ -279,7 +282,7 @@ void b200rwkv_engine::kx_build(const StFile& st, const char* cfg_json, size_t cf
         CK(cudaFuncSetAttribute(latent_attn_tc_kernel<1, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_tc));
         CK(cudaFuncSetAttribute(latent_attn_tc_kernel<2, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_tc));
     }
-    CK(cudaFuncSetAttribute(gla_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    CK(cudaFuncSetAttribute(gla_scan_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SCAN_SMEM));
     CK(cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024));
     REQUIRE(moe_route_smem(W, 2048) <= 128 * 1024, B200RWKV_ERR_UNSUPPORTED, "width too large for the router kernel");
     CK(cudaFuncSetAttribute(lin_tile_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LIN_TC_SMEM));
@@ -301,7 +304,7 @@ void b200rwkv_engine::kx_lin(cudaStream_t s, Profiler* prof, LinParams p, int ro
         int ks = 1;
         if (groups == 1 && !p.off && !p.xlist && p.cnt_gstride == 0)
             while (ks < 8 && ctas * ks * 2 <= 2 * num_sms && nslab / (ks * 2) >= 4 && (size_t)ks * 2 * rows * p.N <= kx->lin_ws_floats) ks *= 2;
-        if (ks > 1) { p.ksplit = ks; p.ws = kx->lin_ws; }
+        if (ks > 1) { p.ksplit = ks; p.ws = s == kx->side_stream && kx->lin_ws_side ? kx->lin_ws_side : kx->lin_ws; }
         launch_k(lin_tile_kernel<false>, dim3(cdiv(p.N, LIN_BN) * ks, cdiv(rows, LIN_BM), groups), dim3(LIN_THREADS), LIN_TC_SMEM, p, KC_GEMM, s, prof);
         if (ks > 1) launch_k(lin_splitk_finish_kernel, dim3(cdiv(p.N, 512), rows), dim3(256), 0, p, KC_GEMM, s, prof);
     }
@@ -316,6 +319,17 @@ void b200rwkv_engine::kx_short_conv(cudaStream_t s, Profiler* prof, const ShortC
     }
     launch_k(short_conv_kernel, dim3(rows, cb), dim3(256), 0, cp, KC_OTHER, s, prof);
     if (cp.taps > 1) launch_k(conv_commit_kernel, dim3(nslot_grid, cb), dim3(256), 0, cp, KC_OTHER, s, prof);
+}
+
+// gated linear attention of a layer: the recurrence, and the norm over heads that are spread over several CTAs
+void b200rwkv_engine::kx_gla(cudaStream_t s, Profiler* prof, const KxLayer& l, int H_, int dk, int dv, const float* q, const float* k, const float* v,
+                             const float* gate, int ld, float* out, int ldo, int rows, int nslot_grid, bool decode) {
+    SeqModel& m = *kx;
+    const ScanShape sh = scan_shape(dk, dv, 3, decode);
+    GlaParams gp{q, k, v, ld, m.z, H_ * dk, l.gla_state, H_, dk, dv, 1.f / l.c.tau, 1.f / sqrtf((float)dk), sh,
+                 {out, ldo, nullptr, gate, ld, l.norm_w, 0, H_, dv, m.cfg.eps, 1.f, 1, MetaView{d_meta, maxT, S}}};
+    launch_k(decode ? gla_scan_kernel<true> : gla_scan_kernel<false>, dim3(H_ * sh.ncta, nslot_grid), dim3(sh.threads), sh.smem_floats() * 4, gp, KC_WKV, s, prof);
+    if (sh.ncta > 1) launch_k(head_norm_kernel, dim3(rows, cdiv(H_, 4)), dim3(128), 0, gp.norm, KC_LN, s, prof);
 }
 
 void b200rwkv_engine::kx_enqueue_step(cudaStream_t s, int rows, int rrows, bool decode, int nsplit, Profiler* prof) {
@@ -335,15 +349,19 @@ void b200rwkv_engine::kx_enqueue_step(cudaStream_t s, int rows, int rrows, bool 
     {
         PageUpdateParams pu{m.sm, m.d_table, m.npages};
         launch_k(page_update_kernel, dim3(1), dim3(128), 0, pu, KC_OTHER, s, prof);
-        EmbedRowsParams ep{m.embed, m.x, W, mv, m.cfg.embed_scale, m.streams};
+        EmbedRowsParams ep{m.embed, m.x, W, mv, m.cfg.embed_scale, m.streams, m.pairs, m.cfg.pair_buckets, m.cfg.pair_mul_prev, m.cfg.pair_mul_cur,
+                           m.sm.tok_pos(), m.last_tok, decode ? 1 : 0};
         launch_k(embed_rows_kernel, dim3(rows), dim3(NORM_THREADS), 0, ep, KC_LN, s, prof);
+        if (m.pairs && !decode) launch_k(last_token_commit_kernel, dim3(cdiv(std::min(S, rows), 128)), dim3(128), 0, ep, KC_LN, s, prof);
     }
     const int nslot_grid = std::min(S, rows);
     // these end with the last norm
-    const bool own_stack = m.cfg.family == KX_FAMILY_ZUFULIX || m.cfg.family == KX_FAMILY_PASOPEL || m.cfg.family == KX_FAMILY_PANUPEL;
+    const bool own_stack = m.cfg.family == KX_FAMILY_ZUFULIX || m.cfg.family == KX_FAMILY_PASOPEL || m.cfg.family == KX_FAMILY_PANUPEL ||
+                           m.cfg.family == KX_FAMILY_FUFIPEL;
     if (m.cfg.family == KX_FAMILY_ZUFULIX) zf_enqueue_layers(s, rows, nslot_grid, decode, nsplit, prof);
     if (m.cfg.family == KX_FAMILY_PASOPEL) ps_enqueue_layers(s, rows, nslot_grid, decode, nsplit, prof);
     if (m.cfg.family == KX_FAMILY_PANUPEL) pn_enqueue_layers(s, rows, nslot_grid, decode, nsplit, prof);
+    if (m.cfg.family == KX_FAMILY_FUFIPEL) ff_enqueue_layers(s, rows, nslot_grid, decode, nsplit, prof);
     for (size_t li = 0; li < m.layers.size() && !own_stack; ++li) {
         KxLayer& l = m.layers[li];
         const KxLayerCfg& c = l.c;
@@ -404,9 +422,8 @@ void b200rwkv_engine::kx_enqueue_step(cudaStream_t s, int rows, int rrows, bool 
             const int H_ = c.heads, dk = c.dim, dv = c.vdim;
             kx_lin(s, prof, lin(m.hs, W, l.proj, m.pr, l.proj_n, l.proj_n, W), rows, 1);
             kx_lin(s, prof, lin(m.pr + 2 * H_ * dk + 2 * H_ * dv, l.proj_n, l.a2, m.z, H_ * dk, H_ * dk, l.a_rank, LE_STORE, l.a2_b), rows, 1);
-            GlaParams gp{m.pr, m.pr + H_ * dk, m.pr + 2 * H_ * dk, m.pr + 2 * H_ * dk + H_ * dv, l.proj_n, m.z, H_ * dk, l.gla_state, m.vout, H_ * dv,
-                         l.norm_w, H_, dk, dv, 1.f / c.tau, 1.f / sqrtf((float)dk), m.cfg.eps, mv};
-            launch_k(gla_kernel, dim3(H_, nslot_grid), dim3(rup(dv, 32)), gla_smem_bytes(dk, dv), gp, KC_WKV, s, prof);
+            kx_gla(s, prof, l, H_, dk, dv, m.pr, m.pr + H_ * dk, m.pr + 2 * H_ * dk, m.pr + 2 * H_ * dk + H_ * dv, l.proj_n, m.vout, H_ * dv, rows, nslot_grid,
+                   decode);
             LinParams po = lin(m.vout, H_ * dv, l.o, m.x, W, W, H_ * dv, LE_GATED_ADD);
             po.gate = m.G; po.ldg = GW;
             kx_lin(s, prof, po, rows, 1);
@@ -506,7 +523,8 @@ void b200rwkv_engine::kx_fill_step(int* hm, const std::vector<int>& slots, const
     if (m.cfg.family != KX_FAMILY_KEMIRAX) {               // CTAs per attention chunk (a cluster): the keys a chunk can see, in tiles
         int seen = 0;
         for (const KxLayer& l : m.layers) {
-            if (l.c.mixer == KX_WINDOW) seen = std::max(seen, std::min(ctx_max, l.c.window + l.c.keep_first + QB));
+            if (l.c.mixer == KX_WINDOW || l.c.mixer == KX_BIAS_WINDOW) seen = std::max(seen, std::min(ctx_max, l.c.window + l.c.keep_first + QB));
+            if (l.c.mixer == KX_CHUNK_GLA) seen = std::max(seen, std::min(ctx_max, l.c.chunk + QB));
             if (l.c.mixer == KX_BIASED || l.c.mixer == KX_PARALLEL) seen = std::max(seen, ctx_max);
             if (m.cfg.family == KX_FAMILY_PASOPEL)         // the window, and one row per block of older tokens
                 seen = std::max(seen, std::min(ctx_max, l.c.window + QB) + (l.c.pool > 0 ? ctx_max / l.c.pool : 0));

@@ -15,8 +15,9 @@
 //                            FMA.
 //
 // Epilogues (fused): bias, sigmoid / silu / erf-gelu / squared relu / capped tanh, a sigmoid gate on the output, accumulate-into-residual
-// (plain or through a gate), and the gated units
-// (clamped, or plain silu(g) * u) on interleaved (gate, up) output pairs.
+// (plain, times a constant, or through a gate), the gated units (clamped, or plain silu(g) * u) on interleaved (gate, up) output pairs,
+// and a split row: plain outputs first, gated units relu(g) * u behind them (a mixer's projections and a feed-forward that read the
+// same input in one launch).
 #pragma once
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -35,6 +36,8 @@ enum LinEpi {
     LE_ADD = 7,         // Y += acc + bias                 (residual accumulate; every element has one writer)
     LE_MUL_SIGMOID = 8, // Y = (acc + bias) * sigmoid(gate[r, n])   (group g reads gate + g * gate_gstride)
     LE_TANH_CAP = 9,    // Y = limit * tanh((acc + bias) / limit)
+    LE_ADD_MUL = 10,    // Y += limit * (acc + bias)       (residual accumulate; every element has one writer)
+    LE_SPLIT_GLU_RELU = 11, // outputs below `split` (even): Y = acc; pairs (split + 2i, split + 2i + 1) = (g, u): Y2[r, i] = max(g, 0) * u
 };
 
 struct LinParams {
@@ -48,7 +51,7 @@ struct LinParams {
     const float* bias;                                 // [N] (nullptr: none); group g adds g * N
     const float* gate; int ldg;                        // LE_GATED_ADD, LE_MUL_SIGMOID
     long long gate_gstride;                            // LE_MUL_SIGMOID: gate + g * gate_gstride
-    float limit;                                       // LE_GLU_CLAMP, LE_TANH_CAP
+    float limit;                                       // LE_GLU_CLAMP, LE_TANH_CAP, LE_ADD_MUL
     int epi;
     int max_rows;                                      // upper bound of any group's rows (grid sizing)
     // split-k (tensor-core tile kernel, one group): blockIdx.x = split * n_tiles + n_tile, split s multiplies its own range of
@@ -56,6 +59,8 @@ struct LinParams {
     // Projections with few output tiles (low-rank stages) otherwise occupy a handful of SMs, each waiting on its own loads.
     int ksplit;                                        // 0 / 1: off
     float* ws;
+    int split;                                         // LE_SPLIT_GLU_RELU
+    float* Y2; int ldy2;
 };
 
 __device__ __forceinline__ float lin_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
@@ -77,6 +82,10 @@ __device__ __forceinline__ void lin_store(const LinParams& p, int g, int yrow, i
         Y[(size_t)yrow * p.ldy + (n >> 1)] = a0 * lin_sigmoid(a0) * a1;
         return;
     }
+    if (p.epi == LE_SPLIT_GLU_RELU && n >= p.split) {
+        p.Y2[(size_t)yrow * p.ldy2 + ((n - p.split) >> 1)] = fmaxf(a0, 0.f) * a1;
+        return;
+    }
     const float* b = p.bias ? p.bias + (size_t)g * p.N : nullptr;
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -90,6 +99,7 @@ __device__ __forceinline__ void lin_store(const LinParams& p, int g, int yrow, i
         else if (p.epi == LE_RELU_SQ) { const float r = fmaxf(a, 0.f); *y = r * r; }
         else if (p.epi == LE_GATED_ADD) *y += p.gate[(size_t)yrow * p.ldg + nn] * a;
         else if (p.epi == LE_ADD) *y += a;
+        else if (p.epi == LE_ADD_MUL) *y += p.limit * a;
         else if (p.epi == LE_MUL_SIGMOID) *y = a * lin_sigmoid(p.gate[g * p.gate_gstride + (size_t)yrow * p.ldg + nn]);
         else if (p.epi == LE_TANH_CAP) *y = p.limit * tanhf(a / p.limit);
         else *y = a;

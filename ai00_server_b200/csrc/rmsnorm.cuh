@@ -1,5 +1,8 @@
 // Root-mean-square normalisation stages on f32 rows (every norm of this family is computed in 32-bit):
-//   embed_rows_kernel      x[t] = table[token[t]] * scale, written to every copy of the residual   (bf16 table -> f32 residual)
+//   embed_rows_kernel      x[t] = table[token[t]] * scale, written to every copy of the residual   (bf16 table -> f32 residual);
+//                          optionally plus a row looked up by a hash of (previous token, token), the previous token being part of
+//                          a sequence's memory
+//   last_token_commit_kernel   the last token of every sequence in the step becomes its previous token
 //   norm_shift_kernel      h = x / rms(x) * g (one scalar gain);  hs = h + (h_prev - h) * mu  (token shift on the NORMED row;
 //                          h_prev = the previous token's h: the row before it in this step, or the sequence's shift state);
 //   shift_commit_kernel    the last token of every sequence in the step leaves its h as the new shift state
@@ -39,17 +42,47 @@ struct EmbedRowsParams {
     MetaView meta;
     float scale = 1.f;       // factor on the row
     int copies = 1;          // the row is written `copies` times: x is [T][copies][W]
+    // pair table (nullptr: none): row (prev * mul_prev + token * mul_cur) mod buckets, row `buckets` for a sequence's first token
+    const __nv_bfloat16* pairs = nullptr;
+    int buckets = 0, mul_prev = 0, mul_cur = 0;
+    const int* pos = nullptr;         // [T] position of the token in its sequence
+    float* last_tok = nullptr;        // [S] the sequence's last token
+    int commit = 0;                   // steps of one token per sequence: the kernel also replaces last_tok
 };
 
 __global__ void __launch_bounds__(NORM_THREADS) embed_rows_kernel(const EmbedRowsParams p) {
     const int t = blockIdx.x;
     if (t >= p.meta.T()) return;
-    const __nv_bfloat16* src = p.table + (size_t)p.meta.tok()[t] * p.W;
+    const int tok = p.meta.tok()[t];
+    const __nv_bfloat16* src = p.table + (size_t)tok * p.W;
+    const __nv_bfloat16* src2 = nullptr;
+    if (p.pairs) {
+        float* last = p.last_tok + p.meta.tok_slot()[t];
+        long long row = p.buckets;
+        if (p.pos[t] > 0) {
+            const int before = p.meta.tok_prev()[t];
+            const long long prev = before >= 0 ? p.meta.tok()[before] : (int)*last;
+            row = (prev * p.mul_prev + (long long)tok * p.mul_cur) % p.buckets;
+        }
+        src2 = p.pairs + row * p.W;
+        if (p.commit) {
+            __syncthreads();                       // every thread has read the old token
+            if (threadIdx.x == 0) *last = (float)tok;
+        }
+    }
     float* dst = p.x + (size_t)t * p.copies * p.W;
     for (int c = threadIdx.x; c < p.W; c += blockDim.x) {
-        const float v = __bfloat162float(src[c]) * p.scale;
+        float v = __bfloat162float(src[c]) * p.scale;
+        if (src2) v += __bfloat162float(src2[c]);
         for (int s = 0; s < p.copies; ++s) dst[(size_t)s * p.W + c] = v;
     }
+}
+
+// own launch after embed_rows_kernel: a first token of the step may still be reading the old one
+__global__ void __launch_bounds__(128) last_token_commit_kernel(const EmbedRowsParams p) {
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= p.meta.nslots()) return;
+    p.last_tok[p.meta.slot_id()[i]] = (float)p.meta.tok()[p.meta.slot_start()[i] + p.meta.slot_count()[i] - 1];
 }
 
 struct NormShiftParams {
@@ -202,13 +235,14 @@ __global__ void __launch_bounds__(NORM_THREADS) norm_add_kernel(const NormAddPar
 // The boundary in front of a pre-norm sublayer.  In this order, each part optional:
 //   x[t] += sum_k wgt[t, k] rows[row_of[t, k]] + shared[t]     the routed feed-forward that just finished (its combine step)
 //   x[t] += post_mul * y[t] / rms(y[t]) * post_w               the sublayer that just finished, with a norm on its output
+//         + post_mul * y2[t] / rms(y2[t]) * post2_w            (two mixers side by side: each output has its own norm)
 //   snap[t] = x[t]                                             the residual as the finished layer leaves it (bring-up aid)
 //   x[t] += table[token[t]] + vec                              a pass of a looped run of layers begins
 //   cat[t] = [x[t]; table[token[t]]]                           a pass begins with a projection of both (then table adds nothing to x)
 //   h[t] = x[t] / rms(x[t]) * weight                           the sublayer's input; `weight` holds the whole factor (a model
 //                                                              that stores offsets from one uploads 1 + w)
 // With `compact` only the rows that want logits are normed and land in h[row]; `hidden` gets a copy of every residual row.
-// All f32.  Dynamic shared memory: W floats.
+// All f32.  Dynamic shared memory: W floats (2 W with y2).
 struct PreNormParams {
     float* x;                 // [T, W] residual, updated in place
     const float* rows;        // [T * top, W] expert outputs in compact rows (nullptr: nothing pending)
@@ -228,6 +262,8 @@ struct PreNormParams {
     const float* post_w = nullptr;    // [W]
     float post_mul = 1.f;
     float* cat = nullptr;             // [T, 2 W] (nullptr: none)
+    const float* y2 = nullptr;        // [T, W] a second output (nullptr: none; only beside y)
+    const float* post2_w = nullptr;   // [W]
 };
 
 constexpr int PRE_NORM_THREADS_FEW_ROWS = 1024;    // block size for steps of few tokens (decode): a thread then owns one or two columns
@@ -248,7 +284,7 @@ __global__ void __launch_bounds__(THREADS) pre_norm_kernel(const PreNormParams p
     }
     const __nv_bfloat16* er = p.table ? p.table + (size_t)p.meta.tok()[t] * W : nullptr;
     const bool writes = p.rows || p.y || (er && !p.cat) || p.vec;
-    float ss = 0.f, post_r = 0.f;
+    float ss = 0.f, post_r = 0.f, post2_r = 0.f;
     if (p.y) {
         for (int c = threadIdx.x; c < W; c += blockDim.x) {        // a thread meets the same columns again below
             const float v = p.y[(size_t)t * W + c];
@@ -259,9 +295,20 @@ __global__ void __launch_bounds__(THREADS) pre_norm_kernel(const PreNormParams p
         post_r = p.post_mul / sqrtf(ss / (float)W + p.eps);
         ss = 0.f;
     }
+    if (p.y2) {
+        for (int c = threadIdx.x; c < W; c += blockDim.x) {
+            const float v = p.y2[(size_t)t * W + c];
+            pre_norm_row[W + c] = v;
+            ss = fmaf(v, v, ss);
+        }
+        ss = rms_block_sum(ss, red);
+        post2_r = p.post_mul / sqrtf(ss / (float)W + p.eps);
+        ss = 0.f;
+    }
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
         float v = xr[c];
         if (p.y) v += pre_norm_row[c] * post_r * p.post_w[c];
+        if (p.y2) v += pre_norm_row[W + c] * post2_r * p.post2_w[c];
         if (p.rows) {
             float f = 0.f;
 #pragma unroll

@@ -1,23 +1,25 @@
-// Softmax attention over a paged cache with a sliding window, a learned "sink" term per head in the softmax denominator, and
-// (optionally) block means of the keys / values that have left the window.  No positions enter the scores here: a layer that
-// rotates its queries and keys does so before it calls this (rot_prep_kernel).
+// Softmax attention over a paged cache with a sliding window and / or inside chunks of the sequence; optionally with a learned "sink"
+// term per head in the softmax denominator, block means of the keys / values that have left the window, the sequence's first tokens
+// kept beside the window, and a learned bias per (distance, head).  Otherwise no positions enter the scores here: a layer that rotates
+// its queries and keys does so before it calls this (rot_prep_kernel).
 //
 // H query heads, G key / value heads (query head h reads head h / (H / G)).  A cache row of D floats holds, for every key /
 // value head c, a key of dk floats at `koff + c dk` and a value of dv floats at `voff + c dv` (the two may be the same floats:
 // a latent row that is scored against and summed, G = 1).  For query position i:
-//     tokens   j with  i - win < j <= i
+//     tokens   j with  low(i) <= j <= i,   low(i) = max(i - win + 1, the first position of i's chunk)     (chunk = 0: one chunk)
+//              and j < keep                                                          (keep > 0: only without blocks)
 //     blocks   b with  (b + 1) pool <= i - win + 1      (pool > 0): the mean of the cache rows b pool .. b pool + pool - 1,
 //              kept in a second pool of rows with the same layout (pool_write_kernel) so that a block costs one row to read
-//     s_h(i, u) = (q_h(i) . k(u)) * scale           over the visible tokens and blocks u together
+//     s_h(i, u) = (q_h(i) . k(u)) * scale  [+ bias[h][min(i - u, nb)]]          over the visible tokens and blocks u together
 //     o_h(i) = sum_u exp(s_h(i, u)) v(u) / (exp(sink_h) + sum_u exp(s_h(i, u)))        * sigmoid(gate_h(i)) * out_mul
 // The gate is optional: one number per output entry, or one per head.
 //
 //   pool_write_kernel     every token of the step that closes a block writes the block's mean row (sums in position order, f32)
 //   pool_rebuild_kernel   the same for all closed blocks of one sequence (after a state import)
-//   rot_prep_kernel       queries and keys of a layer that norms the whole projection and rotates half against half
+//   rot_prep_kernel       queries and keys of a layer that norms the whole projection, rotates half against half, or both
 //   sink_attn_kernel      a cluster of 1..8 CTAs per (chunk of consecutive tokens of one sequence, group of HB query heads);
-//                         the visible block rows and then the window's token rows form 32-key tiles that are dealt out among
-//                         the cluster's CTAs; every CTA walks its tiles once with a running maximum / sum per (token, head) row
+//                         the visible block rows (or kept first tokens) and then the window's token rows form 32-key tiles that
+//                         are dealt out among the cluster's CTAs; every CTA walks its tiles once with a running maximum / sum per (token, head) row
 //                         and the partial results are merged through distributed shared memory in rank order, where the sink
 //                         and the gate come in.  A warp owns 1, 2 or 4 rows of one key / value head (template).  Tiles arrive
 //                         by cp.async into one or two buffers.  Scores, weights and sums in f32.  Any head size.
@@ -77,8 +79,9 @@ __global__ void __launch_bounds__(128) pool_rebuild_kernel(const PoolWriteParams
 
 // Queries and keys of an attention layer that norms each projection as a whole and rotates half against half: per token
 //     q <- rot(q / rms(q over all heads) * w_q) -> step buffer,   k <- rot(k / rms(k over all heads) * w_k) and v -> the cache row
-// where entry i of a head turns with entry i + dims / 2 (i < dims / 2) by position * freq[i] and entries from dims on stay.  One CTA
-// per token; the angles are formed and reduced in double, once per token.  Dynamic shared memory: dims floats.
+// where entry i of a head turns with entry i + dims / 2 (i < dims / 2) by position * freq[i], cosine and sine times mag, and entries
+// from dims on stay.  Without wq (and wk) nothing is normed; without k only the queries are prepared (a layer that reads another
+// layer's cache).  One CTA per token; the angles are formed and reduced in double, once per token.  Dynamic shared memory: dims floats.
 struct RotPrepParams {
     const float* q; const float* k; const float* v; int ld;      // projection rows: q [H dk], k [G dk], v [G dv]
     float* qo; int ldq;                            // [T, H dk]
@@ -89,6 +92,7 @@ struct RotPrepParams {
     int H, G, dk, dv, dims;
     float eps;
     MetaView meta; SeqMeta sm;
+    float mag = 1.f;
 };
 
 constexpr int ROT_PREP_THREADS = 256;
@@ -100,33 +104,44 @@ __global__ void __launch_bounds__(ROT_PREP_THREADS) rot_prep_kernel(const RotPre
     if (t >= p.meta.T()) return;
     const int slot = p.meta.tok_slot()[t], ipos = p.sm.tok_pos()[t], half = p.dims >> 1;
     float* row = p.cache + sa_token_row(p.table + (size_t)slot * p.stride, p.page, ipos) * (size_t)(p.G * (p.dk + p.dv));
-    for (int i = threadIdx.x; i < half; i += blockDim.x) rot_cos_sin(ipos, p.freq[i], rot_cs[i], rot_cs[half + i]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float cs, sn;
+        rot_cos_sin(ipos, p.freq[i], cs, sn);
+        rot_cs[i] = cs * p.mag; rot_cs[half + i] = sn * p.mag;
+    }
     const float* qs = p.q + (size_t)t * p.ld;
     const float* ks = p.k + (size_t)t * p.ld;
     const float* vs = p.v + (size_t)t * p.ld;
-    const int nq = p.H * p.dk, nk = p.G * p.dk;
-    float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < nq; i += blockDim.x) sq = fmaf(qs[i], qs[i], sq);
-    for (int i = threadIdx.x; i < nk; i += blockDim.x) sk = fmaf(ks[i], ks[i], sk);
-    sq = rms_block_sum(sq, red);
-    sk = rms_block_sum(sk, red);                   // its barriers also publish the angles
-    const float rq = 1.f / sqrtf(sq / (float)nq + p.eps), rk = 1.f / sqrtf(sk / (float)nk + p.eps);
+    const bool norm = p.wq != nullptr;
+    const int nq = p.H * p.dk, nk = p.k ? p.G * p.dk : 0;
+    float rq = 1.f, rk = 1.f;
+    if (norm) {
+        float sq = 0.f, sk = 0.f;
+        for (int i = threadIdx.x; i < nq; i += blockDim.x) sq = fmaf(qs[i], qs[i], sq);
+        for (int i = threadIdx.x; i < nk; i += blockDim.x) sk = fmaf(ks[i], ks[i], sk);
+        sq = rms_block_sum(sq, red);
+        sk = rms_block_sum(sk, red);
+        rq = 1.f / sqrtf(sq / (float)nq + p.eps);
+        rk = 1.f / sqrtf(sk / (float)max(nk, 1) + p.eps);
+    }
+    __syncthreads();                               // the angles are there
     for (int e = threadIdx.x; e < nq + nk; e += blockDim.x) {
         const bool isq = e < nq;
         const int o = isq ? e : e - nq, i = o % p.dk;
         const float* src = isq ? qs : ks;
         const float* w = isq ? p.wq : p.wk;
         const float r = isq ? rq : rk;
-        float val = src[o] * r * w[o];
+        float val = norm ? src[o] * r * w[o] : src[o];
         if (i < p.dims) {
             const int f = i < half ? i : i - half, o2 = i < half ? o + half : o - half;
-            const float other = src[o2] * r * w[o2];
+            const float other = norm ? src[o2] * r * w[o2] : src[o2];
             val = i < half ? val * rot_cs[f] - other * rot_cs[half + f] : val * rot_cs[f] + other * rot_cs[half + f];
         }
         if (isq) p.qo[(size_t)t * p.ldq + o] = val;
         else row[o] = val;
     }
-    for (int i = threadIdx.x; i < p.G * p.dv; i += blockDim.x) row[nk + i] = vs[i];
+    if (p.k)
+        for (int i = threadIdx.x; i < p.G * p.dv; i += blockDim.x) row[nk + i] = vs[i];
 }
 
 struct SinkAttnParams {
@@ -149,8 +164,26 @@ struct SinkAttnParams {
     int valias;                                    // the value is the first dv floats of the key (one tile serves both)
     int nsub;                                      // the step's chunks hold nsub * qb tokens: a CTA group takes one part of a chunk
     int ks;                                        // register form: warps of a CTA that share one item's key tiles
+    int keep, chunk;                               // kept first tokens (not beside blocks); tokens per chunk of the sequence (0: none)
+    const float* bias; int nb;                     // [H][nb + 1] added to the scores (nullptr: none; not beside blocks)
     MetaView meta; SeqMeta sm;
 };
+
+// the first position of the window / chunk of query position i
+__device__ __forceinline__ int sa_low(const SinkAttnParams& p, int i) {
+    return max(i - p.win + 1, p.chunk > 0 ? i - i % p.chunk : 0);
+}
+// what the queries pos0 .. pos1 can see: n0 rows of segment 0 (the blocks its last token sees, or the kept tokens in front of the
+// first token's window), then the tokens jlo .. pos1
+__device__ __forceinline__ void sa_segments(const SinkAttnParams& p, int pos0, int pos1, int& n0, int& jlo) {
+    jlo = max(0, sa_low(p, pos0));
+    if (p.pool > 0) {
+        n0 = max(0, pos1 - p.win + 1) / p.pool;
+    } else {
+        n0 = min(p.keep, jlo);
+        if (n0 == jlo) n0 = jlo = 0;               // the kept tokens reach the window: one run
+    }
+}
 
 // which part of which chunk this CTA group works on; false: nothing (the same answer in every CTA of a cluster)
 __device__ __forceinline__ bool sa_chunk(const SinkAttnParams& p, int grp, int& t0, int& nq) {
@@ -206,9 +239,9 @@ __global__ void __launch_bounds__(SA_THREADS) sink_attn_kernel(const SinkAttnPar
     }
     for (int e = threadIdx.x; e < R * dv; e += (int)blockDim.x) sO[e] = 0.f;
     for (int e = threadIdx.x; e < R; e += (int)blockDim.x) { sMax[e] = -CUDART_INF_F; sSum[e] = 0.f; sScl[e] = 1.f; }
-    // what the chunk can see: the blocks its last token sees, then the tokens from the first token's window edge on
-    const int npb = p.pool > 0 ? max(0, pos1 - p.win + 1) / p.pool : 0;
-    const int jlo = max(0, pos0 - p.win + 1), ntk = pos1 - jlo + 1;
+    int npb, jlo;
+    sa_segments(p, pos0, pos1, npb, jlo);
+    const int ntk = pos1 - jlo + 1;
     const int npt = (npb + SA_KT - 1) / SA_KT, ntiles = npt + (ntk + SA_KT - 1) / SA_KT;
     const int* tbl = p.table + (size_t)slot * p.stride;
     const int nrg = nq * nhc;                      // rows of one key / value head
@@ -219,9 +252,9 @@ __global__ void __launch_bounds__(SA_THREADS) sink_attn_kernel(const SinkAttnPar
     const int nstage = rank < ntiles ? ((ntiles - rank + CL - 1) / CL) * ngrp : 0;
     auto load_stage = [&](int rd) {
         const int ti = rank + (rd / ngrp) * CL, g0 = (rd % ngrp) * p.gt, gn = min(p.gt, ncv - g0);
-        const bool pooled = ti < npt;
-        const int i0 = pooled ? ti * SA_KT : jlo + (ti - npt) * SA_KT;          // first block / position of the tile
-        const int nk = pooled ? min(SA_KT, npb - i0) : min(SA_KT, pos1 + 1 - i0);
+        const bool seg0 = ti < npt, pooled = seg0 && p.pool > 0;
+        const int i0 = seg0 ? ti * SA_KT : jlo + (ti - npt) * SA_KT;            // first block / position of the tile
+        const int nk = seg0 ? min(SA_KT, npb - i0) : min(SA_KT, pos1 + 1 - i0);
         float* tk = sK + (size_t)(rd % p.nbuf) * bufK;
         float* tv = sV + (size_t)(rd % p.nbuf) * bufV;
         const size_t offk = (size_t)p.koff + (size_t)(c_first + g0) * dk, offv = (size_t)p.voff + (size_t)(c_first + g0) * dv;
@@ -265,9 +298,9 @@ __global__ void __launch_bounds__(SA_THREADS) sink_attn_kernel(const SinkAttnPar
         __syncthreads();                           // stage rd's tiles are visible (and, the first time, the rows are initialised)
         {
             const int ti = rank + (rd / ngrp) * CL, g0 = (rd % ngrp) * p.gt, gn = min(p.gt, ncv - g0);
-            const bool pooled = ti < npt;
-            const int i0 = pooled ? ti * SA_KT : jlo + (ti - npt) * SA_KT;
-            const int nk = pooled ? min(SA_KT, npb - i0) : min(SA_KT, pos1 + 1 - i0);
+            const bool seg0 = ti < npt, pooled = seg0 && p.pool > 0;
+            const int i0 = seg0 ? ti * SA_KT : jlo + (ti - npt) * SA_KT;
+            const int nk = seg0 ? min(SA_KT, npb - i0) : min(SA_KT, pos1 + 1 - i0);
             const int il = i0 + lane;              // this lane's block or position
             const float* cK = sK + (size_t)(rd % p.nbuf) * bufK;
             const float* cV = valias ? cK : sV + (size_t)(rd % p.nbuf) * bufV;
@@ -313,8 +346,12 @@ __global__ void __launch_bounds__(SA_THREADS) sink_attn_kernel(const SinkAttnPar
                 for (int b = 0; b < RBT; ++b) {
                     if (b >= nr) break;
                     const int r = rows[b], pq = pos0 + r / nh;
-                    const bool vis = lane < nk && (pooled ? il < max(0, pq - p.win + 1) / p.pool : (il <= pq && il > pq - p.win));
-                    const float s = vis ? sc[b] * p.scale : -CUDART_INF_F;
+                    const bool vis = lane < nk && (pooled ? il < max(0, pq - p.win + 1) / p.pool : (il <= pq && (il >= sa_low(p, pq) || il < p.keep)));
+                    float s = -CUDART_INF_F;
+                    if (vis) {
+                        s = sc[b] * p.scale;
+                        if (p.bias) s += p.bias[(size_t)(h0 + r % nh) * (p.nb + 1) + min(pq - il, p.nb)];
+                    }
                     float mx = s;
 #pragma unroll
                     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -422,7 +459,7 @@ __global__ void __launch_bounds__(SA_THREADS) sink_attn_kernel(const SinkAttnPar
 //   scores   eight keys at a time: every lane loads its 16 bytes of each 512-byte piece of a key row straight from the cache,
 //            multiplies them with its query entries, and a butterfly over the lanes (keep half of the keys, send the other
 //            half: 4 + 2 + 1 exchanges, then two plain ones) leaves the finished score of key (l >> 2) of the batch in lane l;
-//   softmax  window / block mask, running maximum / sum with three exchanges per row;
+//   softmax  window / chunk / block mask and bias, running maximum / sum with three exchanges per row;
 //   values   the weight of each key is broadcast from its lane, every lane loads its 16 bytes of each piece of the value row.
 // With few (head, row block) items per chunk the tiles are split over KS warps per item as well as over the cluster's CTAs;
 // the partial (maximum, sum, output) triples meet in shared memory (within a CTA) and then through distributed shared memory
@@ -459,8 +496,9 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
     float* sM2 = sL + (size_t)ncv_cap * nblk_cap * KS * RB;        // [ncv * nblk_cap][RB] merged over the CTA's key splits
     float* sL2 = sM2 + (size_t)ncv_cap * nblk_cap * RB;
     const int* tbl = p.table + (size_t)slot * p.stride;
-    const int npb = p.pool > 0 ? max(0, pos1 - p.win + 1) / p.pool : 0;
-    const int jlo = max(0, pos0 - p.win + 1), ntk = pos1 - jlo + 1;
+    int npb, jlo;
+    sa_segments(p, pos0, pos1, npb, jlo);
+    const int ntk = pos1 - jlo + 1;
     const int npt = (npb + SA_KT - 1) / SA_KT, ntiles = npt + (ntk + SA_KT - 1) / SA_KT;
     const int l4 = lane * 4, kq = lane >> 2;
     const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -483,9 +521,9 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
         }
         const size_t koffs = (size_t)p.koff + (size_t)c * dk + l4, voffs = (size_t)p.voff + (size_t)c * dv + l4;
         for (int ti = rank * KS + ks; ti < ntiles; ti += CL * KS) {
-            const bool pooled = ti < npt;
-            const int i0 = pooled ? ti * SA_KT : jlo + (ti - npt) * SA_KT;
-            const int nk = pooled ? min(SA_KT, npb - i0) : min(SA_KT, pos1 + 1 - i0);
+            const bool seg0 = ti < npt, pooled = seg0 && p.pool > 0;
+            const int i0 = seg0 ? ti * SA_KT : jlo + (ti - npt) * SA_KT;
+            const int nk = seg0 ? min(SA_KT, npb - i0) : min(SA_KT, pos1 + 1 - i0);
             const float* base = pooled ? p.pcache : p.cache;
             unsigned long long myoff = 0ull;                       // row offset of key i0 + lane
             if (lane < nk) myoff = (unsigned long long)(pooled ? sa_pool_row(tbl, p.page, p.pool, p.prow, i0 + lane) : sa_token_row(tbl, p.page, i0 + lane)) * (unsigned)D;
@@ -544,12 +582,14 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
             for (int b = 0; b < RB; ++b) {
                 const int pq = pos0 + qi[b];
                 const int lim = pooled ? max(0, pq - p.win + 1) / p.pool : 0;      // blocks this row sees
+                const int low = sa_low(p, pq);
+                const float* bias = p.bias ? p.bias + (size_t)hh[b] * (p.nb + 1) : nullptr;
                 float tmax = -CUDART_INF_F;
 #pragma unroll
                 for (int bt = 0; bt < 4; ++bt) {
                     const int kk = bt * 8 + kq, i = i0 + kk;
-                    const bool vis = kk < nk && (pooled ? i < lim : (i <= pq && i > pq - p.win));
-                    s[bt][b] = vis ? s[bt][b] * p.scale : -CUDART_INF_F;
+                    const bool vis = kk < nk && (pooled ? i < lim : (i <= pq && (i >= low || i < p.keep)));
+                    s[bt][b] = vis ? s[bt][b] * p.scale + (bias ? bias[min(pq - i, p.nb)] : 0.f) : -CUDART_INF_F;
                     tmax = fmaxf(tmax, s[bt][b]);
                 }
                 tmax = fmaxf(tmax, __shfl_xor_sync(0xffffffffu, tmax, 16));

@@ -17,7 +17,8 @@ static inline SaShape sa_shape(const KxLayerCfg& c) {
     return {c.heads, c.kv_heads, c.dim, c.vdim, false};
 }
 
-static inline bool sa_layer(const KxLayerCfg& c) { return c.mixer == KX_SINK || c.mixer == KX_LATENT || c.mixer == KX_PARALLEL; }
+static inline bool sa_layer(const KxLayerCfg& c) { return c.mixer == KX_SINK || c.mixer == KX_LATENT || c.mixer == KX_PARALLEL ||
+                                                         c.mixer == KX_BIAS_WINDOW || c.mixer == KX_CHUNK_GLA; }
 
 // query heads per CTA: whole key heads, or a part of one key head's query heads; about `want`
 static inline int sa_heads_per_cta(int H, int G, int want) {

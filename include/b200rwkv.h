@@ -122,6 +122,7 @@ typedef struct {
 #define B200RWKV_ARCH_ZUFULIX 102
 #define B200RWKV_ARCH_PASOPEL 103
 #define B200RWKV_ARCH_PANUPEL 104
+#define B200RWKV_ARCH_FUFIPEL 105
 #define B200RWKV_QUANT_NONE 0
 #define B200RWKV_QUANT_INT8 1         /* blocks of 128 inputs: f16 (min, max) + 8-bit codes */
 #define B200RWKV_QUANT_NF4 2          /* blocks of 64 inputs: f16 absmax + 4-bit NormalFloat codes */
