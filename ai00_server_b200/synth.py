@@ -754,3 +754,84 @@ def make_panupel(layers: list, width: int = 64, vocab: int = 96, eps: float = 1e
     bits = {k: to_bf16_bits(np.asarray(v, np.float32).reshape(np.shape(v))) for k, v in t.items()}
     rounded = {k: (b.astype(np.uint32) << 16).view(np.float32).reshape(np.shape(t[k])).astype(np.float64) for k, b in bits.items()}
     return json.dumps(cfg).encode(), pack_st_bf16(t), rounded
+
+
+# ----------------------------------------------------------------------------------------------------------------------
+# Fufipel family (config.json + bf16 safetensors): random weights for tests and bench.py
+# ----------------------------------------------------------------------------------------------------------------------
+def fufipel_layer(kind: str, *, heads=4, kv_heads=None, dim=16, vdim=None, scale=None, window=8, keep_first=2, bias_max=40, kv_from=None, chunk=11,
+                  rot_dims=None, base=10000.0, scaling=None, gla_heads=2, gla_dim=12, gla_vdim=None, tau=16.0, ff=48) -> dict:
+    """One entry of config['layers'].  kind: 'attention' | 'parallel'; ff None: no feed-forward; scaling: (factor, fast, slow, original) or None."""
+    a = {"heads": heads, "kv_heads": int(kv_heads or heads), "dim": dim, "vdim": int(vdim or dim), "scale": float(scale if scale is not None else dim ** -0.5)}
+    if kind == "attention":
+        mixer = {**a, "bias_max": bias_max, "mask": {"size": int(window), "keep_first": int(keep_first)}}
+        if kv_from is not None:
+            mixer["kv_from"] = int(kv_from)
+    elif kind == "parallel":
+        rot = {"base": float(base), "dims": int(dim if rot_dims is None else rot_dims)}
+        if scaling:
+            rot["scaling"] = dict(zip(("factor", "fast", "slow", "original"), scaling))
+        mixer = {"left": {**a, "mask": {"size": int(chunk)}, "rot": rot},
+                 "right": {"heads": gla_heads, "dim": gla_dim, "vdim": int(gla_vdim or gla_dim), "tau": float(tau)}}
+    else:
+        raise ValueError(kind)
+    return {"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": int(ff)} if ff else None}
+
+
+def make_fufipel(layers: list, width: int = 64, vocab: int = 96, eps: float = 1e-5, seed: int = 0, residual_mult: float = 0.6, embed_scale: float = 3.0,
+                 bigram: tuple | None = (61, 17, 5), logit_scale: float = 1.5, rel_rows: int = 12, low_rank: int = 8, arrays: bool = True):
+    """(config.json bytes, safetensors image, dict of float64 arrays holding the bf16-rounded values, or None when `arrays` is
+    off) for a random model of the family.  bigram: (buckets, mul_prev, mul_cur) or None; rel_rows: rows of the distance-bias tables."""
+    rng = np.random.default_rng(seed)
+    W = width
+    t = {}
+
+    def mat(n, k, g=1.0):
+        return (rng.standard_normal((n, k)) * (g / np.sqrt(k))).astype(np.float32)
+
+    def norm(name, n=W, centre=1.0):
+        t[name] = (rng.uniform(0.5, 1.5, n) - 1.0 + centre).astype(np.float32)
+
+    t["embed"] = (rng.standard_normal((vocab, W)) / embed_scale).astype(np.float32)
+    if bigram is not None:
+        t["bigram"] = (rng.standard_normal((bigram[0] + 1, W)) * 0.7).astype(np.float32)
+    for i, l in enumerate(layers):
+        p, m = "l%d." % i, l["mixer"]
+        norm(p + "norm1", centre=0.0)
+        if l["type"] == "attention":
+            H, G, dk, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            q = p + "mix."
+            t[q + "q"] = mat(H * dk, W)
+            norm(q + "q.norm", H * dk)
+            if m.get("kv_from") is None:
+                t[q + "k"], t[q + "v"] = mat(G * dk, W), mat(G * dv, W)
+                norm(q + "k.norm", G * dk)
+            t[q + "rel"] = rng.standard_normal((rel_rows, H)).astype(np.float32)
+            t[q + "g"], t[q + "o"] = mat(H * dv, W, 2.0), mat(W, H * dv, 2.0)
+        else:
+            a, b = m["left"], m["right"]
+            H, G, dk, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            q = p + "mix.left."
+            t[q + "q"], t[q + "k"], t[q + "v"], t[q + "o"] = mat(H * dk, W), mat(G * dk, W), mat(G * dv, W), mat(W, H * dv)
+            norm(q + "out")
+            H, dk, dv = b["heads"], b["dim"], b["vdim"]
+            q = p + "mix.right."
+            t[q + "q"], t[q + "k"], t[q + "v"], t[q + "g"] = mat(H * dk, W), mat(H * dk, W), mat(H * dv, W), mat(H * dv, W, 2.0)
+            t[q + "a1"], t[q + "a2"] = mat(low_rank, W), mat(H * dk, low_rank, 2.0)
+            t[q + "a2.b"] = rng.uniform(-3.0, 4.0, H * dk).astype(np.float32)
+            norm(q + "norm", dv)
+            t[q + "o"] = mat(W, H * dv)
+            norm(q + "out")
+        f = l.get("mlp")
+        if f:
+            t[p + "mlp.gate"], t[p + "mlp.up"], t[p + "mlp.down"] = mat(f["ff"], W, 2.0), mat(f["ff"], W, 2.0), mat(W, f["ff"])
+    norm("final.norm", centre=0.0)
+    cfg = {"architecture": "Fufipel", "embedding": {"scale": float(embed_scale)}, "layers": layers, "logit_scale": float(logit_scale), "norm": {"eps": eps},
+           "residual_mult": float(residual_mult), "vocab": vocab, "width": W}
+    if bigram is not None:
+        cfg["embedding"]["bigram"] = dict(zip(("buckets", "mul_prev", "mul_cur"), (int(v) for v in bigram)))
+    if not arrays:
+        return json.dumps(cfg).encode(), pack_st_bf16(t), None
+    bits = {k: to_bf16_bits(np.asarray(v, np.float32).reshape(np.shape(v))) for k, v in t.items()}
+    rounded = {k: (b.astype(np.uint32) << 16).view(np.float32).reshape(np.shape(t[k])).astype(np.float64) for k, b in bits.items()}
+    return json.dumps(cfg).encode(), pack_st_bf16(t), rounded
