@@ -597,36 +597,90 @@ PN_SIZES = {
 }
 
 
+def _panupel_arm(args, name, time_arm, hbm, tf, peak_kind):
+    """One JSON record: the four-layer Panupel stack (delta rule, attention beside a matrix memory, delta rule, attention beside a
+    matrix memory, all with dense feed-forwards; the two middle layers form a loop that runs once)."""
+    from ai00_server_b200 import runtime, synth
+    B, ctx = args.batch, args.context
+    L = synth.panupel_layer
+    z = PN_SIZES[name]
+    W, V, H, G, dk, dv, ff = z["width"], z["vocab"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["dense_ff"]
+    Hm, mk, mv = z["mm_heads"], z["mm_dim"], z["mm_vdim"]
+    hd = dict(heads=H, kv_heads=G, dim=dk, vdim=dv, ff=ff)
+    par = dict(base=5e5, scaling=(8.0, 1.0, 4.0, 8192), mm_heads=Hm, mm_dim=mk, mm_vdim=mv, **hd)
+    layers = [L("delta", conv=z["conv"], **hd), L("parallel", **par), L("delta", conv=z["conv"], **hd), L("parallel", **par)]
+    cfg, st, _ = synth.make_panupel(layers, width=W, vocab=V, seed=1, loop=(1, 3, 1), arrays=False)
+    # algorithmic work: weights one token touches (a decode step streams the same ones), recurrent states read and written, cache
+    # rows of the whole context in the two attention layers
+    mix_d = 2 * G * dk * W + 2 * H * dv * W + 2 * H * W + W * H * dv
+    mix_p = H * dk * W + G * (dk + dv) * W + H * W + W * H * dv + Hm * (2 * mk + 2 * mv + 2) * W + W * Hm * mv
+    active = 2 * mix_d + 2 * mix_p + 4 * 3 * W * ff + 2 * W * W + V * W
+    state_bytes = 2 * B * (H * dk * dv + Hm * mk * mv) * 4 * 2
+    step_bytes = 2 * active + state_bytes + 2 * B * ctx * G * (dk + dv) * 4
+    attn_flops_tok = 2 * 2 * H * (dk + dv) * ctx / 2 + 2 * 2 * 2 * (H * dk * dv + Hm * mk * mv)     # scores + values, state update + read-out
+    m = runtime.Model(st, max_batch=B, token_chunk_size=512, config=cfg, kv_tokens=B * (ctx + args.warmup + args.steps + 8))
+    r = time_arm(m, V, m.state.reset)
+    m.close()
+    r.update({"family": "panupel", "size": name, "batch": B, "context": ctx, "params_active_per_token": int(active),
+              "decode_algorithmic_bytes_per_step": int(step_bytes),
+              "decode_frac_of_hbm_peak": step_bytes / (r["decode_ms_per_step"] * 1e-3) / (hbm * 1e9),
+              "prefill_tflops": (2 * active + attn_flops_tok) * r["prefill_tokens_per_s"] / 1e12,
+              "prefill_frac_of_bf16_peak": (2 * active + attn_flops_tok) * r["prefill_tokens_per_s"] / 1e12 / tf,
+              "peaks": peak_kind, "dtype": "bf16", "data": "synthetic"})
+    return r
+
+
 def panupel_main(args):
-    """Prefill and decode throughput of the Panupel family (delta rule, attention beside a matrix memory, delta rule, attention beside
-    a matrix memory, all with dense feed-forwards; the two middle layers form a loop that runs once) beside the closest existing
-    family, a Degavik stack of equal width, depth, head counts, head sizes and vocabulary."""
+    """Prefill and decode throughput of the Panupel family beside the closest existing family, a Degavik stack of equal width, depth,
+    head counts, head sizes and vocabulary."""
+    peaks, peak_kind = read_peaks()
+    hbm, tf = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    time_arm = _family_timer(args, np.random.default_rng(7))
+    for name in args.kx_sizes.split(","):
+        print(json.dumps(_panupel_arm(args, name, time_arm, hbm, tf, peak_kind)), flush=True)
+        print(json.dumps(_degavik_arm(args, name, time_arm, hbm, tf, peak_kind)), flush=True)
+
+
+FF_SIZES = {
+    # attention window + kept tokens, bias table rows and the distance of the last bucket, tokens per chunk, gated linear attention heads /
+    # head sizes, rank of its decay projection.  Everything else (width, depth, head counts, head sizes, dense ff, vocabulary) is PN_SIZES'
+    "w1024": dict(window=512, keep_first=4, rel_rows=32, bias_max=512, chunk=4096, gla_heads=4, gla_dim=128, gla_vdim=128, low_rank=16),
+    "w2048": dict(window=512, keep_first=4, rel_rows=32, bias_max=512, chunk=4096, gla_heads=8, gla_dim=128, gla_vdim=128, low_rank=16),
+}
+
+
+def fufipel_main(args):
+    """Prefill and decode throughput of the Fufipel family (windowed attention with a distance bias, chunked attention beside gated
+    linear attention, and the same again, all with dense feed-forwards) beside the closest existing family, a Panupel stack of equal
+    width, depth, head counts, head sizes and vocabulary."""
     from ai00_server_b200 import runtime, synth
     peaks, peak_kind = read_peaks()
     hbm, tf = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
     B, ctx = args.batch, args.context
     time_arm = _family_timer(args, np.random.default_rng(7))
-    L = synth.panupel_layer
+    L = synth.fufipel_layer
     for name in args.kx_sizes.split(","):
-        z = PN_SIZES[name]
-        W, V, H, G, dk, dv, ff = z["width"], z["vocab"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["dense_ff"]
-        Hm, mk, mv = z["mm_heads"], z["mm_dim"], z["mm_vdim"]
+        z = {**PN_SIZES[name], **FF_SIZES[name]}
+        W, V, H, G, dk, dv, ff, rank = z["width"], z["vocab"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["dense_ff"], z["low_rank"]
+        Hg, gk, gv = z["gla_heads"], z["gla_dim"], z["gla_vdim"]
         hd = dict(heads=H, kv_heads=G, dim=dk, vdim=dv, ff=ff)
-        par = dict(base=5e5, scaling=(8.0, 1.0, 4.0, 8192), mm_heads=Hm, mm_dim=mk, mm_vdim=mv, **hd)
-        layers = [L("delta", conv=z["conv"], **hd), L("parallel", **par), L("delta", conv=z["conv"], **hd), L("parallel", **par)]
-        cfg, st, _ = synth.make_panupel(layers, width=W, vocab=V, seed=1, loop=(1, 3, 1), arrays=False)
+        att = L("attention", window=z["window"], keep_first=z["keep_first"], bias_max=z["bias_max"], **hd)
+        par = L("parallel", base=5e5, scaling=(8.0, 32.0, 1.0, 8192), chunk=z["chunk"], gla_heads=Hg, gla_dim=gk, gla_vdim=gv, **hd)
+        cfg, st, _ = synth.make_fufipel([att, par, att, par], width=W, vocab=V, seed=1, bigram=(8191, 31, 7), rel_rows=z["rel_rows"], low_rank=rank,
+                                        arrays=False)
         # algorithmic work: weights one token touches (a decode step streams the same ones), recurrent states read and written, cache
-        # rows of the whole context in the two attention layers
-        mix_d = 2 * G * dk * W + 2 * H * dv * W + 2 * H * W + W * H * dv
-        mix_p = H * dk * W + G * (dk + dv) * W + H * W + W * H * dv + Hm * (2 * mk + 2 * mv + 2) * W + W * Hm * mv
-        active = 2 * mix_d + 2 * mix_p + 4 * 3 * W * ff + 2 * W * W + V * W
-        state_bytes = 2 * B * (H * dk * dv + Hm * mk * mv) * 4 * 2
-        step_bytes = 2 * active + state_bytes + 2 * B * ctx * G * (dk + dv) * 4
-        attn_flops_tok = 2 * 2 * H * (dk + dv) * ctx / 2 + 2 * 2 * 2 * (H * dk * dv + Hm * mk * mv)     # scores + values, state update + read-out
+        # rows inside the window (two layers) and the chunk (two layers)
+        mix_a = H * dk * W + G * (dk + dv) * W + 2 * W * H * dv
+        mix_p = H * dk * W + G * (dk + dv) * W + W * H * dv + Hg * (2 * gk + 2 * gv) * W + W * Hg * gv + rank * (W + Hg * gk)
+        active = 2 * mix_a + 2 * mix_p + 4 * 3 * W * ff + V * W
+        seen = min(ctx, z["window"] + z["keep_first"]) + min(ctx, z["chunk"])
+        seen_mean = min(ctx / 2, z["window"] + z["keep_first"]) + min(ctx, z["chunk"]) / 2
+        step_bytes = 2 * active + 2 * B * Hg * gk * gv * 4 * 2 + 2 * B * seen * G * (dk + dv) * 4
+        attn_flops_tok = 2 * 2 * H * (dk + dv) * seen_mean + 2 * 2 * 2 * Hg * gk * gv      # scores + values, state update + read-out
         m = runtime.Model(st, max_batch=B, token_chunk_size=512, config=cfg, kv_tokens=B * (ctx + args.warmup + args.steps + 8))
         r = time_arm(m, V, m.state.reset)
         m.close()
-        r.update({"family": "panupel", "size": name, "batch": B, "context": ctx, "params_active_per_token": int(active),
+        r.update({"family": "fufipel", "size": name, "batch": B, "context": ctx, "params_active_per_token": int(active),
                   "decode_algorithmic_bytes_per_step": int(step_bytes),
                   "decode_frac_of_hbm_peak": step_bytes / (r["decode_ms_per_step"] * 1e-3) / (hbm * 1e9),
                   "prefill_tflops": (2 * active + attn_flops_tok) * r["prefill_tokens_per_s"] / 1e12,
@@ -634,7 +688,7 @@ def panupel_main(args):
                   "peaks": peak_kind, "dtype": "bf16", "data": "synthetic"})
         print(json.dumps(r), flush=True)
         del st
-        print(json.dumps(_degavik_arm(args, name, time_arm, hbm, tf, peak_kind)), flush=True)
+        print(json.dumps(_panupel_arm(args, name, time_arm, hbm, tf, peak_kind)), flush=True)
 
 
 def main():
@@ -655,10 +709,10 @@ def main():
     ap.add_argument("--quant-layers", type=int, default=-1, help="the reference's `quant`: first N layers (default: all)")
     ap.add_argument("--seqs", type=int, default=256)
     ap.add_argument("--seq-len", type=int, default=512)
-    ap.add_argument("--family", default="rwkv", choices=["rwkv", "kemirax", "degavik", "zufulix", "pasopel", "panupel"],
-                    help="kemirax / degavik / zufulix / pasopel / panupel: prefill and decode throughput of that family at layer sizes of a real model (random "
+    ap.add_argument("--family", default="rwkv", choices=["rwkv", "kemirax", "degavik", "zufulix", "pasopel", "panupel", "fufipel"],
+                    help="kemirax / degavik / zufulix / pasopel / panupel / fufipel: prefill and decode throughput of that family at layer sizes of a real model (random "
                          "weights), beside the closest existing family at equal width and depth (RWKV-7 for kemirax, Kemirax for degavik, "
-                         "Degavik for zufulix, Zufulix for pasopel, Degavik for panupel); one "
+                         "Degavik for zufulix, Zufulix for pasopel, Degavik for panupel, Panupel for fufipel); one "
                          "JSON line per arm (not the headline workload)")
     ap.add_argument("--kx-sizes", default="w1024,w2048", help="--family other than rwkv: comma-separated size names")
     ap.add_argument("--context", type=int, default=1024,
@@ -675,6 +729,8 @@ def main():
         return pasopel_main(args)
     if args.family == "panupel":
         return panupel_main(args)
+    if args.family == "fufipel":
+        return fufipel_main(args)
     PRESET, BATCH = args.preset, args.batch
     METRIC = metric_name(PRESET, BATCH)
     if args.quant != "none":
