@@ -455,12 +455,14 @@ __global__ void __launch_bounds__(SA_THREADS) sink_attn_kernel(const SinkAttnPar
 // ------------------------------------------------------------------------------------------------------------------
 // A warp owns RB rows of one key / value head and a share of the visible tiles, and keeps everything it accumulates in
 // registers: lane l holds entries 128 c + 4 l .. + 3 (c < NC) of the RB query rows and of the RB un-normalised output rows,
-// plus the rows' running maxima and sums.  Per tile of 32 keys:
+// plus the rows' running maxima and sums.  Per tile of 8 NB keys:
 //   scores   eight keys at a time: every lane loads its 16 bytes of each 512-byte piece of a key row straight from the cache,
 //            multiplies them with its query entries, and a butterfly over the lanes (keep half of the keys, send the other
 //            half: 4 + 2 + 1 exchanges, then two plain ones) leaves the finished score of key (l >> 2) of the batch in lane l;
 //   softmax  window / chunk / block mask and bias, running maximum / sum with three exchanges per row;
 //   values   the weight of each key is broadcast from its lane, every lane loads its 16 bytes of each piece of the value row.
+// Prompt steps take tiles of 32 keys (NB = 4: one rescaling per 32).  Decode-shaped steps take tiles of 8 (NB = 1): their few tiles
+// then spread evenly over the warps, the key and value rows of a tile are asked for together, and the code stays short.
 // With few (head, row block) items per chunk the tiles are split over KS warps per item as well as over the cluster's CTAs;
 // the partial (maximum, sum, output) triples meet in shared memory (within a CTA) and then through distributed shared memory
 // (across the cluster), always in a fixed order; the sink term and the gate come in at the end.
@@ -472,8 +474,9 @@ __host__ __device__ inline size_t sink_attn_reg_smem(int qb, int HB, int rep, in
     return (slots * rb * (dv + 2) + 2 * (size_t)ncv * nblk * rb + 8) * sizeof(float);
 }
 
-template <int RB, int NC>
+template <int RB, int NC, int NB>
 __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_kernel(const SinkAttnParams p) {
+    constexpr int KT = 8 * NB;                     // keys per tile
     namespace cg = cooperative_groups;
     cg::cluster_group cluster = cg::this_cluster();
     const int CL = p.cl, rank = blockIdx.x % CL;
@@ -499,7 +502,7 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
     int npb, jlo;
     sa_segments(p, pos0, pos1, npb, jlo);
     const int ntk = pos1 - jlo + 1;
-    const int npt = (npb + SA_KT - 1) / SA_KT, ntiles = npt + (ntk + SA_KT - 1) / SA_KT;
+    const int npt = (npb + KT - 1) / KT, ntiles = npt + (ntk + KT - 1) / KT;
     const int l4 = lane * 4, kq = lane >> 2;
     const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int it = warp; it < ncv * nblk * KS; it += NW) {
@@ -522,15 +525,16 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
         const size_t koffs = (size_t)p.koff + (size_t)c * dk + l4, voffs = (size_t)p.voff + (size_t)c * dv + l4;
         for (int ti = rank * KS + ks; ti < ntiles; ti += CL * KS) {
             const bool seg0 = ti < npt, pooled = seg0 && p.pool > 0;
-            const int i0 = seg0 ? ti * SA_KT : jlo + (ti - npt) * SA_KT;
-            const int nk = seg0 ? min(SA_KT, npb - i0) : min(SA_KT, pos1 + 1 - i0);
+            const int i0 = seg0 ? ti * KT : jlo + (ti - npt) * KT;
+            const int nk = seg0 ? min(KT, npb - i0) : min(KT, pos1 + 1 - i0);
             const float* base = pooled ? p.pcache : p.cache;
             unsigned long long myoff = 0ull;                       // row offset of key i0 + lane
             if (lane < nk) myoff = (unsigned long long)(pooled ? sa_pool_row(tbl, p.page, p.pool, p.prow, i0 + lane) : sa_token_row(tbl, p.page, i0 + lane)) * (unsigned)D;
-            float s[4][RB];
-            // ---- scores: four batches of eight keys ----
+            float s[NB][RB];
+            float4 v0[8];                                          // NB = 1: the first piece of the value rows, asked for with the keys
+            // ---- scores: NB batches of eight keys ----
 #pragma unroll
-            for (int bt = 0; bt < 4; ++bt) {
+            for (int bt = 0; bt < NB; ++bt) {
                 float pt[RB][8];
 #pragma unroll
                 for (int b = 0; b < RB; ++b)
@@ -539,6 +543,10 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
                 unsigned long long off[8];
 #pragma unroll
                 for (int u = 0; u < 8; ++u) off[u] = __shfl_sync(0xffffffffu, myoff, bt * 8 + u);
+                if constexpr (NB == 1) {
+#pragma unroll
+                    for (int u = 0; u < 8; ++u) v0[u] = (l4 < dv && u < nk) ? __ldg(reinterpret_cast<const float4*>(base + off[u] + voffs)) : zero4;
+                }
 #pragma unroll
                 for (int cc = 0; cc < NC; ++cc) {
                     if (128 * cc >= dk) break;                     // warp-uniform
@@ -586,7 +594,7 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
                 const float* bias = p.bias ? p.bias + (size_t)hh[b] * (p.nb + 1) : nullptr;
                 float tmax = -CUDART_INF_F;
 #pragma unroll
-                for (int bt = 0; bt < 4; ++bt) {
+                for (int bt = 0; bt < NB; ++bt) {
                     const int kk = bt * 8 + kq, i = i0 + kk;
                     const bool vis = kk < nk && (pooled ? i < lim : (i <= pq && (i >= low || i < p.keep)));
                     s[bt][b] = vis ? s[bt][b] * p.scale + (bias ? bias[min(pq - i, p.nb)] : 0.f) : -CUDART_INF_F;
@@ -600,7 +608,7 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
                 const float scl = (any && m[b] > -CUDART_INF_F) ? expf(m[b] - mn) : 0.f;
                 float tsum = 0.f;
 #pragma unroll
-                for (int bt = 0; bt < 4; ++bt) {
+                for (int bt = 0; bt < NB; ++bt) {
                     const float w = (any && s[bt][b] > -CUDART_INF_F) ? expf(s[bt][b] - mn) : 0.f;
                     s[bt][b] = w;
                     tsum += w;
@@ -615,13 +623,13 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
             }
             // ---- weights x values ----
 #pragma unroll
-            for (int bt = 0; bt < 4; ++bt) {
+            for (int bt = 0; bt < NB; ++bt) {
                 if (bt * 8 >= nk) break;                           // warp-uniform
                 float w[RB][8];
                 unsigned long long off[8];
 #pragma unroll
                 for (int u = 0; u < 8; ++u) {
-                    off[u] = __shfl_sync(0xffffffffu, myoff, bt * 8 + u);
+                    if (NB > 1 || NC > 1) off[u] = __shfl_sync(0xffffffffu, myoff, bt * 8 + u);
 #pragma unroll
                     for (int b = 0; b < RB; ++b) w[b][u] = __shfl_sync(0xffffffffu, s[bt][b], u << 2);
                 }
@@ -631,8 +639,10 @@ __global__ void __launch_bounds__(SAR_THREADS, NC == 1 ? 2 : 1) sink_attn_reg_ke
                     const bool vact = l4 + 128 * cc < dv;
                     float4 vx[8];
 #pragma unroll
-                    for (int u = 0; u < 8; ++u)
-                        vx[u] = (vact && bt * 8 + u < nk) ? __ldg(reinterpret_cast<const float4*>(base + off[u] + voffs + 128 * cc)) : zero4;
+                    for (int u = 0; u < 8; ++u) {
+                        if (NB == 1 && cc == 0) vx[u] = v0[u];
+                        else vx[u] = (vact && bt * 8 + u < nk) ? __ldg(reinterpret_cast<const float4*>(base + off[u] + voffs + 128 * cc)) : zero4;
+                    }
 #pragma unroll
                     for (int u = 0; u < 8; ++u)
 #pragma unroll

@@ -36,8 +36,9 @@ static inline int sa_heads_per_cta(int H, int G, int want) {
 // the register form is built for key rows of one 512-byte piece per head.  (With three and five pieces, which the kernel's
 // template allows, a decode step of a 576-float latent row took 120 us where the tile form takes 84: every piece's loads wait
 // for the registers of the piece before it.)
-static inline SinkAttnKernel sa_reg_kernel(int rb) {
-    return rb >= 4 ? sink_attn_reg_kernel<4, 1> : (rb == 2 ? sink_attn_reg_kernel<2, 1> : sink_attn_reg_kernel<1, 1>);
+static inline SinkAttnKernel sa_reg_kernel(int rb, bool decode) {
+    if (decode) return rb >= 4 ? sink_attn_reg_kernel<4, 1, 1> : (rb == 2 ? sink_attn_reg_kernel<2, 1, 1> : sink_attn_reg_kernel<1, 1, 1>);
+    return rb >= 4 ? sink_attn_reg_kernel<4, 1, 4> : (rb == 2 ? sink_attn_reg_kernel<2, 1, 4> : sink_attn_reg_kernel<1, 1, 4>);
 }
 
 // how one attention launch of a layer runs: which kernel, its block size and shared memory, and the tile parameters
@@ -55,7 +56,7 @@ static SaPlan sa_plan(const KxLayer& l, int qb_prompt, bool decode) {
         const int items = ncv * cdiv(rows, rb);
         int ks = 1;                                // few items (decode): the 8 warps share each item's key tiles
         while (ks < 8 && items * ks * 2 <= SAR_THREADS / 32) ks *= 2;
-        p.kern = sa_reg_kernel(rb); p.threads = SAR_THREADS; p.smem = sink_attn_reg_smem(qb, HB, rep, a.dv, rb, ks);
+        p.kern = sa_reg_kernel(rb, decode); p.threads = SAR_THREADS; p.smem = sink_attn_reg_smem(qb, HB, rep, a.dv, rb, ks);
         p.gt = 1; p.nbuf = 1; p.qb = qb; p.ks = ks;
         return p;
     }
@@ -121,7 +122,7 @@ static void sa_plan_model(SeqModel& m) {
     if (m.sa_ygroups == 1 << 30) m.sa_ygroups = m.sa_ygroups_decode = 1;       // no attention layer
     for (int rb = 1; rb <= SA_RB; rb *= 2) {
         CK(cudaFuncSetAttribute(sa_tile_kernel(rb), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-        CK(cudaFuncSetAttribute(sa_reg_kernel(rb), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        for (bool decode : {false, true}) CK(cudaFuncSetAttribute(sa_reg_kernel(rb, decode), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     }
     // the largest cluster the attention launch may ask for: what the device can co-schedule at this layer's shared memory
     for (const KxLayer& l : m.layers) {

@@ -27,6 +27,7 @@ constexpr int SCAN_MAX_DK = 32 * SCAN_R;
 constexpr int SCAN_THREADS = 512;                  // most threads per CTA (a whole head at once: steps of one token per sequence)
 constexpr int SCAN_THREADS_PROMPT = 128;
 constexpr int SCAN_SMEM = 64 * 1024;               // most shared memory of a launch
+constexpr int SCAN_SMEM_FIVE = 44 * 1024;          // ... with five CTAs on an SM
 
 struct ScanShape {
     int ks, lks, rt;                               // lanes per column (a power of two and its logarithm), entries per lane (a multiple of 4)
@@ -61,7 +62,8 @@ __host__ inline ScanShape scan_shape(int dk, int dv, int rows, bool decode) {
     s.ncta = (dv + s.cols - 1) / s.cols;
     s.nbuf = decode ? 1 : 2;
     s.tc = decode ? 1 : 16;
-    while (s.tc > 1 && s.smem_floats() * sizeof(float) > SCAN_SMEM) s.tc /= 2;
+    // five CTAs per SM (their registers allow no more): many heads and sequences then still fit one wave
+    while (s.tc > 1 && s.smem_floats() * sizeof(float) > (s.tc > 4 ? SCAN_SMEM_FIVE : SCAN_SMEM)) s.tc /= 2;
     return s;
 }
 

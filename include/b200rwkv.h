@@ -107,7 +107,8 @@ typedef struct {
      * architecture "Pasopel": pre-norm blocks, a run of layers executed several times, windowed attention with block means and
      * a sink term, windowed latent attention, dense or routed feed-forwards; architecture "Panupel": blocks normed on both sides of
      * every sublayer, a run of layers executed several times, attention beside a matrix memory, gated delta rule, dense
-     * feed-forwards; bf16 weights): the JSON text, borrowed during the call.  NULL: the
+     * feed-forwards; architecture "Fufipel": one norm for mixer and feed-forward, windowed attention with a distance bias, chunked
+     * attention beside gated linear attention, pair embeddings; bf16 weights): the JSON text, borrowed during the call.  NULL: the
      * family is recognised from the tensor names (RWKV v5 / v6 / v7).  Such models keep an attention cache in pages of
      * `kv_page` tokens (0 = 64) drawn from a pool sized for `kv_tokens` tokens over all live sequences (0 = 4096 per slot);
      * precision 0 = bf16 tensor-core products with f32 accumulation, 1 = every product in plain f32.  Their steps hold up to
