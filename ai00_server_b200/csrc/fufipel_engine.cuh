@@ -149,7 +149,7 @@ void b200rwkv_engine::ff_enqueue_layers(cudaStream_t s, int rows, int nslot_grid
         LinParams p;
         memset(&p, 0, sizeof(p));
         p.X = X; p.ldx = ldx; p.W = Wt; p.Y = Y; p.ldy = ldy; p.N = N_; p.K = K_; p.cnt = cntT; p.epi = epi; p.bias = bias;
-        p.limit = mul;                             // LE_ADD_MUL: the factor on a sublayer's contribution
+        p.limit = mul;                             // LE_ADD: the factor on a sublayer's contribution
         return p;
     };
     const KxLayer* halves = nullptr;               // a parallel layer whose two outputs wait in m.y and m.hs
@@ -184,7 +184,7 @@ void b200rwkv_engine::ff_enqueue_layers(cudaStream_t s, int rows, int nslot_grid
             kx_lin(s2, prof, lin(m.pr + r.ra, PN, l.a2, m.z, Hr * mk, Hr * mk, l.a_rank, LE_STORE, l.a2_b), rows, 1);
             kx_gla(s2, prof, l, Hr, mk, mvd, m.pr + r.rq, m.pr + r.rk, m.pr + r.rv, m.pr + r.rg, PN, m.vout + r.heads, KO, rows, nslot_grid, decode);
             kx_lin(s2, prof, lin(m.vout + r.heads, KO, l.o2, m.hs, W, W, r.rheads), rows, 1);
-            if (c.has_mlp) kx_lin(s2, prof, lin(m.vout + r.heads + r.rheads, KO, l.sh_down, m.x, W, W, c.ff, LE_ADD_MUL), rows, 1);
+            if (c.has_mlp) kx_lin(s2, prof, lin(m.vout + r.heads + r.rheads, KO, l.sh_down, m.x, W, W, c.ff, LE_ADD), rows, 1);
         }
         const bool own = c.kv_from < 0;
         RotPrepParams rp{m.pr + r.q, own ? m.pr + r.k : nullptr, own ? m.pr + r.v : nullptr, PN, m.q, H_ * dk, l.cache, m.d_table, m.npages, m.page,
@@ -211,7 +211,7 @@ void b200rwkv_engine::ff_enqueue_layers(cudaStream_t s, int rows, int nslot_grid
             kx_lin(s, prof, lin(m.vout, KO, l.o, m.y, W, W, r.heads), rows, 1);
             halves = &l;
         } else {                                   // attention and feed-forward in one product, straight into the residual
-            kx_lin(s, prof, lin(m.vout, KO, l.o, m.x, W, W, KO, LE_ADD_MUL), rows, 1);
+            kx_lin(s, prof, lin(m.vout, KO, l.o, m.x, W, W, KO, LE_ADD), rows, 1);
         }
         if (fork) { CK(cudaEventRecord(m.side_join, s2)); CK(cudaStreamWaitEvent(s, m.side_join, 0)); }
         if (m.dbg_layers && !use_graph)            // bring-up aid: the residual as this layer leaves it

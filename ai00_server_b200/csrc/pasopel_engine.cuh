@@ -159,6 +159,7 @@ void b200rwkv_engine::ps_enqueue_layers(cudaStream_t s, int rows, int nslot_grid
         LinParams p;
         memset(&p, 0, sizeof(p));
         p.X = X; p.ldx = ldx; p.W = Wt; p.Y = Y; p.ldy = ldy; p.N = N_; p.K = K_; p.cnt = cntT; p.epi = epi; p.bias = bias;
+        p.limit = 1.f;                             // LE_ADD adds the product as it is
         return p;
     };
     struct Pending { const float* rows = nullptr; int top = 0; const float* shared = nullptr; };
