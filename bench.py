@@ -666,7 +666,7 @@ def fufipel_main(args):
         hd = dict(heads=H, kv_heads=G, dim=dk, vdim=dv, ff=ff)
         att = L("attention", window=z["window"], keep_first=z["keep_first"], bias_max=z["bias_max"], **hd)
         par = L("parallel", base=5e5, scaling=(8.0, 32.0, 1.0, 8192), chunk=z["chunk"], gla_heads=Hg, gla_dim=gk, gla_vdim=gv, **hd)
-        cfg, st, _ = synth.make_fufipel([att, par, att, par], width=W, vocab=V, seed=1, bigram=(8191, 31, 7), rel_rows=z["rel_rows"], low_rank=rank,
+        cfg, st, _ = synth.make_fufipel([att, par, att, par], width=W, vocab=V, seed=1, bigram=(8191, 131, 53), rel_rows=z["rel_rows"], low_rank=rank,
                                         arrays=False)
         # algorithmic work: weights one token touches (a decode step streams the same ones), recurrent states read and written, cache
         # rows inside the window (two layers) and the chunk (two layers)
